@@ -5,3 +5,4 @@ from .panolorn import PanolornConfig
 from .pevolorn import PevolornConfig
 from .qwen3 import Qwen3Config
 from .tetodra import TetodraConfig
+from .vigonex import VigonexConfig

@@ -6,7 +6,10 @@
 //   a window       keys pos - window + 1 .. pos,
 //   a sink         one more term in the softmax's denominator that carries no value: exp(0), or exp(z_h) with a
 //                  learned number z_h per query head (`sink_logit`; it is not scaled, capped or biased),
-// and after the softmax an output gate: out *= sigmoid(gate).  Values may also be the first dv elements of
+// and, instead of one attention map per head, the difference of two (`MAPS` = 2): a query head and a key head hold two
+// vectors of width dk each, every map is a softmax of its own over the same values, and the head's result is
+// a1 - lambda a2, divided by its root mean square over dv and times a constant (DiffMod);
+// and after that an output gate: out *= sigmoid(gate).  Values may also be the first dv elements of
 // wider rows (`v_row` elements from one value to the next; the attention over compressed vectors that serve
 // as keys and, in part, as values passes the key plane twice).  Every constant is an argument; a
 // zero (or a null pointer) switches its step off, and with all of them off this is plain causal
@@ -45,6 +48,11 @@ __device__ __forceinline__ float dist_bias_of(const ScoreMod& m, int head, int d
     if (m.dist_bias == nullptr) return 0.0f;
     return m.dist_bias[(size_t)head * m.dist_len + min(max(dist, 0), m.dist_len - 1)];
 }
+
+// The difference of two maps: o = a1 - lambda * a2, then o / sqrt(mean(o^2) + eps) * out_scale.
+struct DiffMod {
+    float lambda, eps, out_scale;
+};
 
 static inline int page_shift_of(int page_size) {
     int shift = 0;
@@ -271,19 +279,21 @@ qkv_unit_store_vec_kernel(const bf16* proj, int row_stride, const bf16* __restri
 // ---------------------------------------------------------------- general kernel
 constexpr int kGenWarps = 4;
 
-template <typename T, int CK, int CV>
+template <typename T, int CK, int CV, int MAPS>
 __global__ void attention_biased_general_kernel(
     const T* q, const T* k_plane, const T* v_plane, long long page_stride,
     const int* __restrict__ positions, const int* __restrict__ token_slot,
     const int* __restrict__ block_table, int max_pages, int page_size, int q_heads, int kv_heads,
-    int dk, int dv, ScoreMod mod, const float* __restrict__ slopes, const float* __restrict__ sink_logit, int v_row,
+    int dk, int dv, ScoreMod mod, DiffMod diff, const float* __restrict__ slopes, const float* __restrict__ sink_logit, int v_row,
     const T* gate, int gate_stride, T* __restrict__ out) {
     extern __shared__ float smem[];
+    __shared__ float scratch[32];
     TLLM_PDL_ENTER();
-    float* qs = smem;                             // [dk]
-    float* acc_s = smem + dk;                     // [warps][dv]
-    float* m_s = acc_s + kGenWarps * dv;          // [warps]
-    float* l_s = m_s + kGenWarps;                 // [warps]
+    const int kd = MAPS * dk;                     // elements of a query head and of a cached key
+    float* qs = smem;                             // [MAPS][dk]
+    float* acc_s = smem + kd;                     // [MAPS][warps][dv]
+    float* m_s = acc_s + MAPS * kGenWarps * dv;   // [MAPS][warps]
+    float* l_s = m_s + MAPS * kGenWarps;          // [MAPS][warps]
 
     const int head = blockIdx.x, t = blockIdx.y;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -297,85 +307,121 @@ __global__ void attention_biased_general_kernel(
     const int lo = first_key(pos, mod);
     const int g = head / (q_heads / kv_heads);
     const float slope = slopes != nullptr ? slopes[head] : 0.0f;
-    const T* qsrc = q + ((size_t)t * q_heads + head) * dk;
-    for (int e = threadIdx.x; e < dk; e += blockDim.x) qs[e] = to_f32<T>(qsrc[e]);
+    const T* qsrc = q + ((size_t)t * q_heads + head) * kd;
+    for (int e = threadIdx.x; e < kd; e += blockDim.x) qs[e] = to_f32<T>(qsrc[e]);
     __syncthreads();
 
     const int* table = block_table + (size_t)slot * max_pages;
     // the sink is a key of score 0 (or of the head's learned score) without a value; warp 0 starts from it
-    float m = (mod.sink && warp == 0) ? (sink_logit != nullptr ? sink_logit[head] : 0.0f) : -INFINITY;
-    float l = (mod.sink && warp == 0) ? 1.0f : 0.0f;
-    float acc[CV];
+    float m[MAPS], l[MAPS], acc[MAPS][CV];
 #pragma unroll
-    for (int c = 0; c < CV; ++c) acc[c] = 0.0f;
+    for (int mp = 0; mp < MAPS; ++mp) {
+        m[mp] = (mod.sink && warp == 0) ? (sink_logit != nullptr ? sink_logit[head] : 0.0f) : -INFINITY;
+        l[mp] = (mod.sink && warp == 0) ? 1.0f : 0.0f;
+#pragma unroll
+        for (int c = 0; c < CV; ++c) acc[mp][c] = 0.0f;
+    }
 
     for (int j = lo + warp; j <= pos; j += kGenWarps) {
         const int page = table[j / page_size];
         if (page < 0) continue;
         const size_t in_page = (size_t)g * page_size + (j % page_size);
-        const T* kp = k_plane + (long long)page * page_stride + in_page * dk;
+        const T* kp = k_plane + (long long)page * page_stride + in_page * kd;
         const T* vp = v_plane + (long long)page * page_stride + in_page * v_row;
-        float dot = 0.0f;
 #pragma unroll
-        for (int c = 0; c < CK; ++c) {
-            const int e = lane + 32 * c;
-            if (e < dk) dot += qs[e] * to_f32<T>(kp[e]);
+        for (int mp = 0; mp < MAPS; ++mp) {
+            float dot = 0.0f;
+#pragma unroll
+            for (int c = 0; c < CK; ++c) {
+                const int e = lane + 32 * c;
+                if (e < dk) dot += qs[mp * dk + e] * to_f32<T>(kp[mp * dk + e]);
+            }
+            dot = warp_sum(dot);
+            const float s = mod_score(dot, slope, pos - j, mod) + dist_bias_of(mod, head, pos - j);
+            const float m_new = fmaxf(m[mp], s);
+            const float corr = expf(m[mp] - m_new);
+            const float p = expf(s - m_new);
+            l[mp] = l[mp] * corr + p;
+#pragma unroll
+            for (int c = 0; c < CV; ++c) {
+                const int e = lane + 32 * c;
+                if (e < dv) acc[mp][c] = acc[mp][c] * corr + p * to_f32<T>(vp[e]);
+            }
+            m[mp] = m_new;
         }
-        dot = warp_sum(dot);
-        const float s = mod_score(dot, slope, pos - j, mod) + dist_bias_of(mod, head, pos - j);
-        const float m_new = fmaxf(m, s);
-        const float corr = expf(m - m_new);
-        const float p = expf(s - m_new);
-        l = l * corr + p;
+    }
+#pragma unroll
+    for (int mp = 0; mp < MAPS; ++mp) {
+        if (lane == 0) { m_s[mp * kGenWarps + warp] = m[mp]; l_s[mp * kGenWarps + warp] = l[mp]; }
 #pragma unroll
         for (int c = 0; c < CV; ++c) {
             const int e = lane + 32 * c;
-            if (e < dv) acc[c] = acc[c] * corr + p * to_f32<T>(vp[e]);
+            if (e < dv) acc_s[(mp * kGenWarps + warp) * dv + e] = acc[mp][c];
         }
-        m = m_new;
-    }
-    if (lane == 0) { m_s[warp] = m; l_s[warp] = l; }
-#pragma unroll
-    for (int c = 0; c < CV; ++c) {
-        const int e = lane + 32 * c;
-        if (e < dv) acc_s[warp * dv + e] = acc[c];
     }
     __syncthreads();
-    float mm = m_s[0];
+    float w_scale[MAPS][kGenWarps];               // a warp's share of a map's result, its sum divided out
 #pragma unroll
-    for (int w = 1; w < kGenWarps; ++w) mm = fmaxf(mm, m_s[w]);
-    float w_scale[kGenWarps], total = 0.0f;
+    for (int mp = 0; mp < MAPS; ++mp) {
+        float mm = m_s[mp * kGenWarps], total = 0.0f;
 #pragma unroll
-    for (int w = 0; w < kGenWarps; ++w) {
-        w_scale[w] = (m_s[w] == -INFINITY) ? 0.0f : expf(m_s[w] - mm);
-        total += l_s[w] * w_scale[w];
+        for (int w = 1; w < kGenWarps; ++w) mm = fmaxf(mm, m_s[mp * kGenWarps + w]);
+#pragma unroll
+        for (int w = 0; w < kGenWarps; ++w) {
+            w_scale[mp][w] = (m_s[mp * kGenWarps + w] == -INFINITY) ? 0.0f : expf(m_s[mp * kGenWarps + w] - mm);
+            total += l_s[mp * kGenWarps + w] * w_scale[mp][w];
+        }
+        const float inv = total > 0.0f ? 1.0f / total : 0.0f;
+        if (MAPS > 1) {
+#pragma unroll
+            for (int w = 0; w < kGenWarps; ++w) w_scale[mp][w] *= mp == 0 ? inv : -diff.lambda * inv;
+        } else {
+            m[0] = inv;                           // one map: the sum over the warps is taken first
+        }
     }
-    const float inv = total > 0.0f ? 1.0f / total : 0.0f;
+    float norm = 1.0f;
+    if (MAPS > 1) {
+        float sum = 0.0f;
+        for (int e = threadIdx.x; e < dv; e += blockDim.x) {
+            float v = 0.0f;
+#pragma unroll
+            for (int mp = 0; mp < MAPS; ++mp)
+#pragma unroll
+                for (int w = 0; w < kGenWarps; ++w) v += acc_s[(mp * kGenWarps + w) * dv + e] * w_scale[mp][w];
+            acc_s[e] = v;                         // only this thread looks at column e
+            sum += v * v;
+        }
+        norm = diff.out_scale / sqrtf(block_sum(sum, scratch) / (float)dv + diff.eps);
+    }
     const T* grow = gate != nullptr ? gate + (size_t)t * gate_stride + gate_at(mod.gate_per_head, head, dv, 0) : nullptr;
     for (int e = threadIdx.x; e < dv; e += blockDim.x) {
         float v = 0.0f;
+        if (MAPS > 1) {
+            v = acc_s[e] * norm;
+        } else {
 #pragma unroll
-        for (int w = 0; w < kGenWarps; ++w) v += acc_s[w * dv + e] * w_scale[w];
-        v *= inv;
+            for (int w = 0; w < kGenWarps; ++w) v += acc_s[w * dv + e] * w_scale[0][w];
+            v *= m[0];
+        }
         if (grow != nullptr) v *= 1.0f / (1.0f + expf(-to_f32<T>(grow[mod.gate_per_head ? 0 : e])));
         dst[e] = from_f32<T>(v);
     }
 }
 
-template <typename T>
+template <typename T, int MAPS>
 static int launch_general(const void* q, const void* kp, const void* vp, long long page_stride,
                           const int* positions, const int* token_slot, const int* block_table,
                           int max_pages, int page_size, int tokens, int q_heads, int kv_heads, int dk,
-                          int dv, ScoreMod mod, const float* slopes, const float* sink_logit, int v_row,
+                          int dv, ScoreMod mod, DiffMod diff, const float* slopes, const float* sink_logit, int v_row,
                           const void* gate, int gate_stride, void* out, cudaStream_t stream) {
     const dim3 grid(q_heads, tokens), block(kGenWarps * 32);
-    const size_t smem = ((size_t)dk + (size_t)kGenWarps * dv + 2 * kGenWarps) * sizeof(float);
+    const size_t smem = (size_t)MAPS * ((size_t)dk + (size_t)kGenWarps * dv + 2 * kGenWarps) * sizeof(float);
     const int ck = (dk + 31) / 32, cv = (dv + 31) / 32;
     const int c = ck > cv ? ck : cv;
 #define LAUNCH(C)                                                                                           \
-    launch_pdl(kPdlAttention, attention_biased_general_kernel<T, C, C>, grid, block, smem, stream,          \
+    launch_pdl(kPdlAttention, attention_biased_general_kernel<T, C, C, MAPS>, grid, block, smem, stream,          \
                (const T*)q, (const T*)kp, (const T*)vp, page_stride, positions, token_slot, block_table,    \
-               max_pages, page_size, q_heads, kv_heads, dk, dv, mod, slopes, sink_logit, v_row, (const T*)gate, gate_stride, (T*)out)
+               max_pages, page_size, q_heads, kv_heads, dk, dv, mod, diff, slopes, sink_logit, v_row, (const T*)gate, gate_stride, (T*)out)
     if (c <= 1) LAUNCH(1);
     else if (c <= 2) LAUNCH(2);
     else if (c <= 4) LAUNCH(4);
@@ -426,31 +472,37 @@ __device__ __forceinline__ float mod_score_fast(float dot, float slope_log2e, fl
 // can see in tiles of 64 (flash-attention style: S and the softmax in float32 registers, P V accumulated
 // in float32).  Keys and values are staged by cp.async in two buffers; a row of a tile is padded by 16
 // bytes so that ldmatrix meets no bank conflict, and widths below DKP / DVP are filled with zeros.
+// With two maps a block owns 32 query rows: two of its warps hold them for the first map, two for the second, all
+// share the tiles (a key row holds both maps' keys), and the maps meet in shared memory at the end.
 constexpr int kPfWarps = 4, kPfM = 64, kPfN = 64, kPfPad = 8;
 
-template <int DKP, int DVP>
+template <int DKP, int DVP, int MAPS>
 __global__ void __launch_bounds__(kPfWarps * 32, 3)
 attention_biased_prefill_kernel(const bf16* q, const bf16* k_plane, const bf16* v_plane, long long page_stride,
                                 const int* __restrict__ seg_info, const int* __restrict__ tiles,
                                 const int* __restrict__ block_table, int max_pages, int page_size,
-                                int page_shift, int q_heads, int kv_heads, int dk, int dv, ScoreMod mod,
+                                int page_shift, int q_heads, int kv_heads, int dk, int dv, ScoreMod mod, DiffMod diff,
                                 const float* __restrict__ slopes, const float* __restrict__ sink_logit, int v_row,
                                 const bf16* gate, int gate_stride, bf16* __restrict__ out) {
     extern __shared__ __align__(128) unsigned char pf_smem[];
     TLLM_PDL_ENTER();
-    constexpr int kKRow = DKP + kPfPad, kVRow = DVP + kPfPad;           // elements per padded row
+    constexpr int kKRow = MAPS * DKP + kPfPad, kVRow = DVP + kPfPad;    // elements per padded row
     constexpr int kKBytes = kPfN * kKRow * 2, kVBytes = kPfN * kVRow * 2;
-    const int seg = tiles[2 * blockIdx.x], q_off = tiles[2 * blockIdx.x + 1];
+    constexpr int kRows = kPfM / MAPS, kMapWarps = kPfWarps / MAPS;     // query rows of the block, warps per map
+    const int kd = MAPS * dk;                                           // elements of a query head and of a cached key
+    const int seg = tiles[2 * blockIdx.x], q_off = tiles[2 * blockIdx.x + 1] + (MAPS > 1 ? (int)blockIdx.z * kRows : 0);
     const int head = blockIdx.y;
     const int slot = seg_info[4 * seg], start = seg_info[4 * seg + 1];
     const int len = seg_info[4 * seg + 2], pos0 = seg_info[4 * seg + 3];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (MAPS > 1 && q_off >= len) return;                               // the second half of a block of 64 rows may be empty
+    const int lane = threadIdx.x & 31, map = (threadIdx.x >> 5) / kMapWarps;
+    const int warp = (threadIdx.x >> 5) % kMapWarps;                    // among the warps of the map
     const int g = head / (q_heads / kv_heads);
     const int* table = block_table + (size_t)slot * max_pages;
     const float slope2 = (slopes != nullptr ? slopes[head] : 0.0f) * kLog2e;
     const float inv_cap = mod.softcap > 0.0f ? 1.0f / mod.softcap : 0.0f;
 
-    const int rows_here = min(kPfM, len - q_off);
+    const int rows_here = min(kRows, len - q_off);
     const int first_pos = pos0 + q_off, last_pos = first_pos + rows_here - 1;
     const int lo_all = first_key(first_pos, mod);
     const int kt_first = lo_all / kPfN, kt_last = last_pos / kPfN;
@@ -459,8 +511,8 @@ attention_biased_prefill_kernel(const bf16* q, const bf16* k_plane, const bf16* 
     const bool v_lo = r_lo < rows_here, v_hi = r_hi < rows_here;
     const int p_lo = first_pos + r_lo, p_hi = first_pos + r_hi;
     const int f_lo = first_key(p_lo, mod), f_hi = first_key(p_hi, mod);
-    const bf16* q_lo = q + ((size_t)(start + q_off + r_lo) * q_heads + head) * dk;
-    const bf16* q_hi = q + ((size_t)(start + q_off + r_hi) * q_heads + head) * dk;
+    const bf16* q_lo = q + ((size_t)(start + q_off + r_lo) * q_heads + head) * kd + map * dk;
+    const bf16* q_hi = q + ((size_t)(start + q_off + r_hi) * q_heads + head) * kd + map * dk;
     uint32_t qa[DKP / 16][4];
 #pragma unroll
     for (int ks = 0; ks < DKP / 16; ++ks) {
@@ -486,7 +538,7 @@ attention_biased_prefill_kernel(const bf16* q, const bf16* k_plane, const bf16* 
     auto issue = [&](int kt, int stage) {
         const uint32_t ks = smem_u32(pf_smem + (size_t)stage * (kKBytes + kVBytes));
         const uint32_t vs = ks + kKBytes;
-        constexpr int kKC = DKP / 8, kVC = DVP / 8;
+        constexpr int kMC = DKP / 8, kKC = MAPS * kMC, kVC = DVP / 8;       // 16-byte pieces of a map's key, a row of keys, a value
         // a thread keeps its 16-byte column and walks the rows: one look-up of the page per row
         for (int row = threadIdx.x / kKC, chunk = threadIdx.x % kKC; row < kPfN; row += kPfWarps * 32 / kKC) {
             const int key = kt * kPfN + row;
@@ -496,8 +548,9 @@ attention_biased_prefill_kernel(const bf16* q, const bf16* k_plane, const bf16* 
             const bool ok = page >= 0;
             const long long page_at = ok ? (long long)page * page_stride : 0;
             const long long in_page = (long long)g * page_size + place;
-            const bool k_ok = ok && chunk * 8 < dk;
-            cp_async_16(ks + (row * kKRow + chunk * 8) * 2, k_plane + (k_ok ? page_at + in_page * dk + chunk * 8 : 0), k_ok);
+            const int in_key = (chunk % kMC) * 8;                       // within its map's key
+            const bool k_ok = ok && in_key < dk;
+            cp_async_16(ks + (row * kKRow + chunk * 8) * 2, k_plane + (k_ok ? page_at + in_page * kd + (chunk / kMC) * dk + in_key : 0), k_ok);
             if (kKC == kVC) {
                 const bool v_ok = ok && chunk * 8 < dv;
                 cp_async_16(vs + (row * kVRow + chunk * 8) * 2, v_plane + (v_ok ? page_at + in_page * v_row + chunk * 8 : 0), v_ok);
@@ -540,7 +593,7 @@ attention_biased_prefill_kernel(const bf16* q, const bf16* k_plane, const bf16* 
 #pragma unroll
                 for (int nt2 = 0; nt2 < kPfN / 16; ++nt2) {
                     uint32_t kb[4];
-                    ldmatrix_x4(kb, ks_base + ((nt2 * 16 + (mid >> 1) * 8 + mrow) * kKRow + ks * 16 + (mid & 1) * 8) * 2);
+                    ldmatrix_x4(kb, ks_base + ((nt2 * 16 + (mid >> 1) * 8 + mrow) * kKRow + map * DKP + ks * 16 + (mid & 1) * 8) * 2);
                     const uint32_t b0[2] = {kb[0], kb[1]}, b1[2] = {kb[2], kb[3]};
                     mma_bf16_16816(s[2 * nt2], qa[ks], b0);
                     mma_bf16_16816(s[2 * nt2 + 1], qa[ks], b1);
@@ -642,8 +695,42 @@ attention_biased_prefill_kernel(const bf16* q, const bf16* k_plane, const bf16* 
     l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
-    const float inv_lo = l_lo > 0.0f ? 1.0f / l_lo : 0.0f, inv_hi = l_hi > 0.0f ? 1.0f / l_hi : 0.0f;
+    float inv_lo = l_lo > 0.0f ? 1.0f / l_lo : 0.0f, inv_hi = l_hi > 0.0f ? 1.0f / l_hi : 0.0f;
     const size_t row_lo = start + q_off + r_lo, row_hi = start + q_off + r_hi;
+    if (MAPS > 1) {
+        // the second map's rows, times lambda, in shared memory (over the tiles, which every warp is done with); the
+        // first map's warps take them off their own, and a row's four lanes add up its squares
+        float* meet = reinterpret_cast<float*>(pf_smem);                 // [kRows][DVP + 2]
+        constexpr int kMeet = DVP + 2;
+        if (map == 1) {
+            const float a_lo = inv_lo * diff.lambda, a_hi = inv_hi * diff.lambda;
+#pragma unroll
+            for (int i = 0; i < DVP / 8; ++i) {
+                const int col = i * 8 + (lane & 3) * 2;
+                *reinterpret_cast<float2*>(meet + r_lo * kMeet + col) = make_float2(o[i][0] * a_lo, o[i][1] * a_lo);
+                *reinterpret_cast<float2*>(meet + r_hi * kMeet + col) = make_float2(o[i][2] * a_hi, o[i][3] * a_hi);
+            }
+        }
+        __syncthreads();
+        if (map == 1) return;
+        float sq_lo = 0.0f, sq_hi = 0.0f;
+#pragma unroll
+        for (int i = 0; i < DVP / 8; ++i) {                              // columns past dv are zeros in both maps
+            const int col = i * 8 + (lane & 3) * 2;
+            const float2 b_lo = *reinterpret_cast<const float2*>(meet + r_lo * kMeet + col);
+            const float2 b_hi = *reinterpret_cast<const float2*>(meet + r_hi * kMeet + col);
+            o[i][0] = o[i][0] * inv_lo - b_lo.x; o[i][1] = o[i][1] * inv_lo - b_lo.y;
+            o[i][2] = o[i][2] * inv_hi - b_hi.x; o[i][3] = o[i][3] * inv_hi - b_hi.y;
+            sq_lo += o[i][0] * o[i][0] + o[i][1] * o[i][1];
+            sq_hi += o[i][2] * o[i][2] + o[i][3] * o[i][3];
+        }
+        sq_lo += __shfl_xor_sync(0xffffffffu, sq_lo, 1);
+        sq_lo += __shfl_xor_sync(0xffffffffu, sq_lo, 2);
+        sq_hi += __shfl_xor_sync(0xffffffffu, sq_hi, 1);
+        sq_hi += __shfl_xor_sync(0xffffffffu, sq_hi, 2);
+        inv_lo = diff.out_scale / sqrtf(sq_lo / (float)dv + diff.eps);
+        inv_hi = diff.out_scale / sqrtf(sq_hi / (float)dv + diff.eps);
+    }
     bf16* o_lo = out + (row_lo * q_heads + head) * dv;
     bf16* o_hi = out + (row_hi * q_heads + head) * dv;
     const bf16* g_lo = gate != nullptr ? gate + row_lo * gate_stride + gate_at(mod.gate_per_head, head, dv, 0) : nullptr;
@@ -672,23 +759,23 @@ attention_biased_prefill_kernel(const bf16* q, const bf16* k_plane, const bf16* 
     }
 }
 
-template <int DKP, int DVP>
+template <int DKP, int DVP, int MAPS>
 static int launch_biased_prefill(const void* q, const void* kp, const void* vp, long long page_stride,
                                  const int* seg_info, const int* tiles, int n_tiles, const int* block_table,
                                  int max_pages, int page_size, int q_heads, int kv_heads, int dk, int dv,
-                                 ScoreMod mod, const float* slopes, const float* sink_logit, int v_row, const void* gate,
+                                 ScoreMod mod, DiffMod diff, const float* slopes, const float* sink_logit, int v_row, const void* gate,
                                  int gate_stride, void* out, cudaStream_t stream) {
-    const size_t smem = (size_t)2 * kPfN * ((DKP + kPfPad) + (DVP + kPfPad)) * 2;
+    const size_t smem = (size_t)2 * kPfN * ((MAPS * DKP + kPfPad) + (DVP + kPfPad)) * 2;
     static OncePerDevice configured;
     if (configured.first()) {
-        cudaError_t e = cudaFuncSetAttribute(attention_biased_prefill_kernel<DKP, DVP>,
+        cudaError_t e = cudaFuncSetAttribute(attention_biased_prefill_kernel<DKP, DVP, MAPS>,
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) { set_error("attention_biased_prefill: %s", cudaGetErrorString(e)); return (int)e; }
         configured.done();
     }
-    launch_pdl(kPdlAttention, attention_biased_prefill_kernel<DKP, DVP>, dim3(n_tiles, q_heads), dim3(kPfWarps * 32),
+    launch_pdl(kPdlAttention, attention_biased_prefill_kernel<DKP, DVP, MAPS>, dim3(n_tiles, q_heads, MAPS), dim3(kPfWarps * 32),
                smem, stream, (const bf16*)q, (const bf16*)kp, (const bf16*)vp, page_stride, seg_info, tiles,
-               block_table, max_pages, page_size, page_shift_of(page_size), q_heads, kv_heads, dk, dv, mod, slopes, sink_logit, v_row,
+               block_table, max_pages, page_size, page_shift_of(page_size), q_heads, kv_heads, dk, dv, mod, diff, slopes, sink_logit, v_row,
                (const bf16*)gate, gate_stride, (bf16*)out);
     return finish_launch("attention_biased_prefill");
 }
@@ -701,18 +788,22 @@ static int launch_biased_prefill(const void* q, const void* kp, const void* vp, 
 // the order of the warps.  With one run per row the block writes the result; with more (a grid that
 // would not fill the GPU, long reaches) it leaves unnormalised sums, maximum and weight per run, and a
 // second kernel adds the runs in their order.  The sink belongs to the first warp of the first run.
-template <int DKP, int DVP>
+// With two maps a tile's rows are the group's heads for the first map, then the same heads for the second; a row's
+// query is its map's half of a vector as wide as a row of keys (both maps' keys side by side), the other half zeros,
+// so that one product serves both maps and keys and values are still read once.
+template <int DKP, int DVP, int MAPS>
 __global__ void __launch_bounds__(kPfWarps * 32, 2)
 attention_biased_decode_kernel(const bf16* q, const bf16* k_plane, const bf16* v_plane, long long page_stride,
                                const int* __restrict__ positions, const int* __restrict__ token_slot,
                                const int* __restrict__ rows, const int* __restrict__ block_table, int max_pages,
                                int page_size, int page_shift, int q_heads, int kv_heads, int dk, int dv, ScoreMod mod,
-                               const float* __restrict__ slopes, const float* __restrict__ sink_logit, int v_row,
+                               DiffMod diff, const float* __restrict__ slopes, const float* __restrict__ sink_logit, int v_row,
                                const bf16* gate, int gate_stride, int splits, int sub_groups, float* part,
                                bf16* __restrict__ out) {
     extern __shared__ __align__(128) unsigned char pf_smem[];
     TLLM_PDL_ENTER();
-    constexpr int kKRow = DKP + kPfPad, kVRow = DVP + kPfPad;
+    constexpr int kKRow = MAPS * DKP + kPfPad, kVRow = DVP + kPfPad;
+    const int kd = MAPS * dk;                                           // elements of a query head and of a cached key
     constexpr int kKBytes = kPfN * kKRow * 2, kVBytes = kPfN * kVRow * 2;
     const int t = rows != nullptr ? rows[blockIdx.x] : blockIdx.x;
     // a key/value head's query heads fill the tile's 16 rows; more of them (multi-query attention over many
@@ -739,21 +830,26 @@ attention_biased_decode_kernel(const bf16* q, const bf16* k_plane, const bf16* v
         kt_last = min(kt_last, kt_first + per - 1);
     }
 
-    const int r_lo = lane >> 2, r_hi = r_lo + 8;                       // rows of the tile: heads of the group
-    const bool v_lo = r_lo < group, v_hi = r_hi < group;
-    const float slope_lo = (slopes != nullptr && v_lo) ? slopes[head0 + r_lo] * kLog2e : 0.0f;
-    const float slope_hi = (slopes != nullptr && v_hi) ? slopes[head0 + r_hi] * kLog2e : 0.0f;
+    const int r_lo = lane >> 2, r_hi = r_lo + 8;                       // rows of the tile: heads of the group (per map)
+    const int used = MAPS * group;
+    const bool v_lo = r_lo < used, v_hi = r_hi < used;
+    const int map_lo = MAPS > 1 && r_lo >= group ? 1 : 0, map_hi = MAPS > 1 && r_hi >= group ? 1 : 0;
+    const int h_lo = r_lo - map_lo * group, h_hi = r_hi - map_hi * group;          // heads of the group that the rows are
+    const float slope_lo = (slopes != nullptr && v_lo) ? slopes[head0 + h_lo] * kLog2e : 0.0f;
+    const float slope_hi = (slopes != nullptr && v_hi) ? slopes[head0 + h_hi] * kLog2e : 0.0f;
     const float inv_cap = mod.softcap > 0.0f ? 1.0f / mod.softcap : 0.0f;
-    const bf16* q_lo = q + ((size_t)t * q_heads + head0 + r_lo) * dk;
-    const bf16* q_hi = q + ((size_t)t * q_heads + head0 + r_hi) * dk;
-    uint32_t qa[DKP / 16][4];
+    const bf16* q_lo = q + ((size_t)t * q_heads + head0 + h_lo) * kd + map_lo * dk;
+    const bf16* q_hi = q + ((size_t)t * q_heads + head0 + h_hi) * kd + map_hi * dk;
+    uint32_t qa[MAPS * DKP / 16][4];
 #pragma unroll
-    for (int ks = 0; ks < DKP / 16; ++ks) {
-        const int c0 = ks * 16 + (lane & 3) * 2;
-        qa[ks][0] = (v_lo && c0 < dk) ? *reinterpret_cast<const uint32_t*>(q_lo + c0) : 0u;
-        qa[ks][1] = (v_hi && c0 < dk) ? *reinterpret_cast<const uint32_t*>(q_hi + c0) : 0u;
-        qa[ks][2] = (v_lo && c0 + 8 < dk) ? *reinterpret_cast<const uint32_t*>(q_lo + c0 + 8) : 0u;
-        qa[ks][3] = (v_hi && c0 + 8 < dk) ? *reinterpret_cast<const uint32_t*>(q_hi + c0 + 8) : 0u;
+    for (int ks = 0; ks < MAPS * DKP / 16; ++ks) {
+        const int mk = ks / (DKP / 16);                                 // the map whose keys these columns are
+        const int c0 = (ks - mk * (DKP / 16)) * 16 + (lane & 3) * 2;
+        const bool w_lo = v_lo && map_lo == mk, w_hi = v_hi && map_hi == mk;
+        qa[ks][0] = (w_lo && c0 < dk) ? *reinterpret_cast<const uint32_t*>(q_lo + c0) : 0u;
+        qa[ks][1] = (w_hi && c0 < dk) ? *reinterpret_cast<const uint32_t*>(q_hi + c0) : 0u;
+        qa[ks][2] = (w_lo && c0 + 8 < dk) ? *reinterpret_cast<const uint32_t*>(q_lo + c0 + 8) : 0u;
+        qa[ks][3] = (w_hi && c0 + 8 < dk) ? *reinterpret_cast<const uint32_t*>(q_hi + c0 + 8) : 0u;
     }
     float o[DVP / 8][4];
 #pragma unroll
@@ -761,15 +857,15 @@ attention_biased_decode_kernel(const bf16* q, const bf16* k_plane, const bf16* v
     const bool first = mod.sink && warp == 0 && split == 0;
     float m_lo = first ? 0.0f : -INFINITY, m_hi = m_lo;
     if (first && sink_logit != nullptr) {            // the heads' learned sink scores, in base 2 like the scores
-        m_lo = v_lo ? sink_logit[head0 + r_lo] * kLog2e : 0.0f;
-        m_hi = v_hi ? sink_logit[head0 + r_hi] * kLog2e : 0.0f;
+        m_lo = v_lo ? sink_logit[head0 + h_lo] * kLog2e : 0.0f;
+        m_hi = v_hi ? sink_logit[head0 + h_hi] * kLog2e : 0.0f;
     }
     float l_lo = (first && (lane & 3) == 0) ? 1.0f : 0.0f, l_hi = l_lo;
 
     auto issue = [&](int kt, int stage) {
         const uint32_t ks = smem_u32(pf_smem + (size_t)stage * (kKBytes + kVBytes));
         const uint32_t vs = ks + kKBytes;
-        constexpr int kKC = DKP / 8, kVC = DVP / 8;
+        constexpr int kMC = DKP / 8, kKC = MAPS * kMC, kVC = DVP / 8;       // 16-byte pieces of a map's key, a row of keys, a value
         for (int row = threadIdx.x / kKC, chunk = threadIdx.x % kKC; row < kPfN; row += kPfWarps * 32 / kKC) {
             const int key = kt * kPfN + row;
             int page_index, place;
@@ -778,8 +874,9 @@ attention_biased_decode_kernel(const bf16* q, const bf16* k_plane, const bf16* v
             const bool ok = page >= 0;
             const long long page_at = ok ? (long long)page * page_stride : 0;
             const long long in_page = (long long)g * page_size + place;
-            const bool k_ok = ok && chunk * 8 < dk;
-            cp_async_16(ks + (row * kKRow + chunk * 8) * 2, k_plane + (k_ok ? page_at + in_page * dk + chunk * 8 : 0), k_ok);
+            const int in_key = (chunk % kMC) * 8;                       // within its map's key
+            const bool k_ok = ok && in_key < dk;
+            cp_async_16(ks + (row * kKRow + chunk * 8) * 2, k_plane + (k_ok ? page_at + in_page * kd + (chunk / kMC) * dk + in_key : 0), k_ok);
             if (kKC == kVC) {
                 const bool v_ok = ok && chunk * 8 < dv;
                 cp_async_16(vs + (row * kVRow + chunk * 8) * 2, v_plane + (v_ok ? page_at + in_page * v_row + chunk * 8 : 0), v_ok);
@@ -816,7 +913,7 @@ attention_biased_decode_kernel(const bf16* q, const bf16* k_plane, const bf16* v
             float s[2][4];
             s[0][0] = s[0][1] = s[0][2] = s[0][3] = s[1][0] = s[1][1] = s[1][2] = s[1][3] = 0.0f;
 #pragma unroll
-            for (int ks = 0; ks < DKP / 16; ++ks) {
+            for (int ks = 0; ks < MAPS * DKP / 16; ++ks) {
                 uint32_t kb[4];
                 ldmatrix_x4(kb, ks_base + ((warp * 16 + (mid >> 1) * 8 + mrow) * kKRow + ks * 16 + (mid & 1) * 8) * 2);
                 const uint32_t b0[2] = {kb[0], kb[1]}, b1[2] = {kb[2], kb[3]};
@@ -836,8 +933,8 @@ attention_biased_decode_kernel(const bf16* q, const bf16* k_plane, const bf16* v
                     float a = mod_score_fast(s[nt][e], slope_lo, dist, mod, inv_cap);
                     float b = mod_score_fast(s[nt][2 + e], slope_hi, dist, mod, inv_cap);
                     if (mod.dist_bias != nullptr) {
-                        a += dist_bias_of(mod, head0 + (v_lo ? r_lo : 0), pos - j) * kLog2e;
-                        b += dist_bias_of(mod, head0 + (v_hi ? r_hi : 0), pos - j) * kLog2e;
+                        a += dist_bias_of(mod, head0 + (v_lo ? h_lo : 0), pos - j) * kLog2e;
+                        b += dist_bias_of(mod, head0 + (v_hi ? h_hi : 0), pos - j) * kLog2e;
                     }
                     s[nt][e] = (seen && v_lo) ? a : -INFINITY;
                     s[nt][2 + e] = (seen && v_hi) ? b : -INFINITY;
@@ -886,36 +983,70 @@ attention_biased_decode_kernel(const bf16* q, const bf16* k_plane, const bf16* v
     l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
-    // the warps meet: [warp][head of the group][dv + 2] floats, over the staging buffers (all reads of which are done)
+    // the warps meet: [warp][row of the tile in use][dv + 2] floats, over the staging buffers (all reads of which are done)
     float* meet = reinterpret_cast<float*>(pf_smem);
 #pragma unroll
     for (int i = 0; i < DVP / 8; ++i) {
         const int col = i * 8 + (lane & 3) * 2;
         if (col >= dv) continue;
-        if (v_lo) { float* d = meet + ((size_t)warp * group + r_lo) * rec; d[col] = o[i][0]; d[col + 1] = o[i][1]; }
-        if (v_hi) { float* d = meet + ((size_t)warp * group + r_hi) * rec; d[col] = o[i][2]; d[col + 1] = o[i][3]; }
+        if (v_lo) { float* d = meet + ((size_t)warp * used + r_lo) * rec; d[col] = o[i][0]; d[col + 1] = o[i][1]; }
+        if (v_hi) { float* d = meet + ((size_t)warp * used + r_hi) * rec; d[col] = o[i][2]; d[col + 1] = o[i][3]; }
     }
     if ((lane & 3) == 0) {
-        if (v_lo) { float* d = meet + ((size_t)warp * group + r_lo) * rec; d[dv] = m_lo; d[dv + 1] = l_lo; }
-        if (v_hi) { float* d = meet + ((size_t)warp * group + r_hi) * rec; d[dv] = m_hi; d[dv + 1] = l_hi; }
+        if (v_lo) { float* d = meet + ((size_t)warp * used + r_lo) * rec; d[dv] = m_lo; d[dv + 1] = l_lo; }
+        if (v_hi) { float* d = meet + ((size_t)warp * used + r_hi) * rec; d[dv] = m_hi; d[dv + 1] = l_hi; }
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < group * dv; i += blockDim.x) {
-        const int h = i / dv, e = i % dv;
-        float mm = -INFINITY;
+    // element e of row h of the tile, added over the warps: its sum, the weights' sum and their maximum (base 2)
+    auto add_warps = [&](int h, int e, float& v, float& total, float& mm) {
+        mm = -INFINITY;
 #pragma unroll
-        for (int w = 0; w < kPfWarps; ++w) mm = fmaxf(mm, meet[((size_t)w * group + h) * rec + dv]);
-        float total = 0.0f, v = 0.0f;
+        for (int w = 0; w < kPfWarps; ++w) mm = fmaxf(mm, meet[((size_t)w * used + h) * rec + dv]);
+        total = v = 0.0f;
 #pragma unroll
         for (int w = 0; w < kPfWarps; ++w) {
-            const float* src = meet + ((size_t)w * group + h) * rec;
+            const float* src = meet + ((size_t)w * used + h) * rec;
             const float wt = src[dv] == -INFINITY ? 0.0f : fast_exp2(src[dv] - mm);
             total += src[dv + 1] * wt;
             v += src[e] * wt;
         }
+    };
+    if (MAPS > 1 && splits == 1) {                    // a warp per head: the difference of its two rows, normed
+        for (int h = warp; h < group; h += kPfWarps) {
+            float d[DVP / 32], sum = 0.0f;
+#pragma unroll
+            for (int c = 0; c < DVP / 32; ++c) {
+                const int e = lane + 32 * c;
+                d[c] = 0.0f;
+                if (e < dv) {
+                    float v1, v2, t1, t2, mm;
+                    add_warps(h, e, v1, t1, mm);
+                    add_warps(group + h, e, v2, t2, mm);
+                    d[c] = (t1 > 0.0f ? v1 / t1 : 0.0f) - diff.lambda * (t2 > 0.0f ? v2 / t2 : 0.0f);
+                }
+                sum += d[c] * d[c];
+            }
+            const float norm = diff.out_scale / sqrtf(warp_sum(sum) / (float)dv + diff.eps);
+#pragma unroll
+            for (int c = 0; c < DVP / 32; ++c) {
+                const int e = lane + 32 * c;
+                if (e >= dv) continue;
+                float v = d[c] * norm;
+                if (gate != nullptr)
+                    v *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)t * gate_stride + gate_at(mod.gate_per_head, head0 + h, dv, e)])));
+                out[((size_t)t * q_heads + head0 + h) * dv + e] = __float2bfloat16_rn(v);
+            }
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < used * dv; i += blockDim.x) {
+        const int h = i / dv, e = i % dv;
+        float mm, total, v;
+        add_warps(h, e, v, total, mm);
         if (splits > 1) {
-            // [row of the grid][head][split][dv + 2]: sums, then maximum (base 2) and weight
-            float* dst = part + (((size_t)blockIdx.x * q_heads + head0 + h) * splits + split) * rec;
+            // [row of the grid][head (, map)][split][dv + 2]: sums, then maximum (base 2) and weight
+            const int map = MAPS > 1 && h >= group ? 1 : 0;
+            float* dst = part + ((((size_t)blockIdx.x * q_heads + head0 + h - map * group) * MAPS + map) * splits + split) * rec;
             dst[e] = v;
             if (e == 0) { dst[dv] = mm; dst[dv + 1] = total; }
             continue;
@@ -927,11 +1058,14 @@ attention_biased_decode_kernel(const bf16* q, const bf16* k_plane, const bf16* v
     }
 }
 
-// The runs of a (row, head) added in their order, the gate applied, the result written.
+// The runs of a (row, head) added in their order (with two maps: of both, then the normed difference), the gate
+// applied, the result written.
+template <int MAPS>
 __global__ void attention_biased_combine_kernel(const float* part, const int* __restrict__ token_slot,
                                                 const int* __restrict__ rows, int q_heads, int dv, int splits,
-                                                const bf16* gate, int gate_stride, int gate_per_head,
+                                                const bf16* gate, int gate_stride, int gate_per_head, DiffMod diff,
                                                 bf16* __restrict__ out) {
+    __shared__ float scratch[32], row_s[MAPS > 1 ? 128 : 1];
     TLLM_PDL_ENTER();
     const int t = rows != nullptr ? rows[blockIdx.x] : blockIdx.x;
     const int head = blockIdx.y, rec = dv + 2;
@@ -940,53 +1074,70 @@ __global__ void attention_biased_combine_kernel(const float* part, const int* __
         for (int e = threadIdx.x; e < dv; e += blockDim.x) dst[e] = __float2bfloat16_rn(0.0f);
         return;
     }
-    const float* src = part + ((size_t)blockIdx.x * q_heads + head) * splits * rec;
-    float mm = -INFINITY;
-    for (int s2 = 0; s2 < splits; ++s2) mm = fmaxf(mm, src[s2 * rec + dv]);
-    for (int e = threadIdx.x; e < dv; e += blockDim.x) {
+    float norm = 1.0f, mm[MAPS];
+    const float* src[MAPS];
+#pragma unroll
+    for (int mp = 0; mp < MAPS; ++mp) {
+        src[mp] = part + (((size_t)blockIdx.x * q_heads + head) * MAPS + mp) * splits * rec;
+        mm[mp] = -INFINITY;
+        for (int s2 = 0; s2 < splits; ++s2) mm[mp] = fmaxf(mm[mp], src[mp][s2 * rec + dv]);
+    }
+    auto added = [&](int mp, int e) -> float {
         float total = 0.0f, v = 0.0f;
         for (int s2 = 0; s2 < splits; ++s2) {
-            const float ms = src[s2 * rec + dv];
-            const float w = ms == -INFINITY ? 0.0f : fast_exp2(ms - mm);
-            total += src[s2 * rec + dv + 1] * w;
-            v += src[s2 * rec + e] * w;
+            const float ms = src[mp][s2 * rec + dv];
+            const float w = ms == -INFINITY ? 0.0f : fast_exp2(ms - mm[mp]);
+            total += src[mp][s2 * rec + dv + 1] * w;
+            v += src[mp][s2 * rec + e] * w;
         }
-        v = total > 0.0f ? v / total : 0.0f;
+        return total > 0.0f ? v / total : 0.0f;
+    };
+    if (MAPS > 1) {
+        float sum = 0.0f;
+        for (int e = threadIdx.x; e < dv; e += blockDim.x) {
+            const float v = added(0, e) - diff.lambda * added(MAPS - 1, e);
+            row_s[e] = v;                             // only this thread looks at element e
+            sum += v * v;
+        }
+        norm = diff.out_scale / sqrtf(block_sum(sum, scratch) / (float)dv + diff.eps);
+    }
+    for (int e = threadIdx.x; e < dv; e += blockDim.x) {
+        float v = MAPS > 1 ? row_s[e] * norm : added(0, e);
         if (gate != nullptr) v *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)t * gate_stride + gate_at(gate_per_head, head, dv, e)])));
         dst[e] = __float2bfloat16_rn(v);
     }
 }
 
 // Blocks that share a key/value head's query heads in the one-token kernel: the fewest that leave each at
-// most the tile's 16 rows and divide the heads evenly; 0 if there is no such number.
-static int biased_sub_groups(int group) {
+// most the tile's 16 rows (`maps` of them per head) and divide the heads evenly; 0 if there is no such number.
+static int biased_sub_groups(int group, int maps) {
     for (int s = 1; s <= group; ++s)
-        if (group % s == 0 && group / s <= 16) return s;
+        if (group % s == 0 && group / s * maps <= 16) return s;
     return 0;
 }
 
-template <int DKP, int DVP>
+template <int DKP, int DVP, int MAPS>
 static int launch_biased_decode(const void* q, const void* kp, const void* vp, long long page_stride,
                                 const int* positions, const int* token_slot, const int* rows, int n_rows,
                                 const int* block_table, int max_pages, int page_size, int q_heads, int kv_heads,
-                                int dk, int dv, ScoreMod mod, const float* slopes, const float* sink_logit, int v_row,
+                                int dk, int dv, ScoreMod mod, DiffMod diff, const float* slopes, const float* sink_logit, int v_row,
                                 const void* gate, int gate_stride, int splits, float* part, void* out, cudaStream_t stream) {
-    const size_t smem = (size_t)2 * kPfN * ((DKP + kPfPad) + (DVP + kPfPad)) * 2;      // also holds the warps' meeting
+    const size_t smem = (size_t)2 * kPfN * ((MAPS * DKP + kPfPad) + (DVP + kPfPad)) * 2;      // also holds the warps' meeting
     static OncePerDevice configured;
     if (configured.first()) {
-        cudaError_t e = cudaFuncSetAttribute(attention_biased_decode_kernel<DKP, DVP>,
+        cudaError_t e = cudaFuncSetAttribute(attention_biased_decode_kernel<DKP, DVP, MAPS>,
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) { set_error("attention_biased_decode: %s", cudaGetErrorString(e)); return (int)e; }
         configured.done();
     }
-    const int sub_groups = biased_sub_groups(q_heads / kv_heads);
-    launch_pdl(kPdlAttention, attention_biased_decode_kernel<DKP, DVP>, dim3(n_rows, kv_heads * sub_groups, splits), dim3(kPfWarps * 32),
+    const int sub_groups = biased_sub_groups(q_heads / kv_heads, MAPS);
+    launch_pdl(kPdlAttention, attention_biased_decode_kernel<DKP, DVP, MAPS>, dim3(n_rows, kv_heads * sub_groups, splits), dim3(kPfWarps * 32),
                smem, stream, (const bf16*)q, (const bf16*)kp, (const bf16*)vp, page_stride, positions, token_slot,
-               rows, block_table, max_pages, page_size, page_shift_of(page_size), q_heads, kv_heads, dk, dv, mod, slopes, sink_logit, v_row,
+               rows, block_table, max_pages, page_size, page_shift_of(page_size), q_heads, kv_heads, dk, dv, mod, diff, slopes, sink_logit, v_row,
                (const bf16*)gate, gate_stride, splits, sub_groups, part, (bf16*)out);
     if (splits > 1)
-        launch_pdl(kPdlCombine, attention_biased_combine_kernel, dim3(n_rows, q_heads), dim3(dv >= 128 ? 128 : 64), 0, stream,
-                   (const float*)part, token_slot, rows, q_heads, dv, splits, (const bf16*)gate, gate_stride, mod.gate_per_head, (bf16*)out);
+        launch_pdl(kPdlCombine, attention_biased_combine_kernel<MAPS>, dim3(n_rows, q_heads), dim3(dv >= 128 ? 128 : 64), 0, stream,
+                   (const float*)part, token_slot, rows, q_heads, dv, splits, (const bf16*)gate, gate_stride, mod.gate_per_head, diff, (bf16*)out);
     return finish_launch("attention_biased_decode");
 }
 
@@ -1049,8 +1200,11 @@ int tllm_attention_biased_general(
     const void* q, const void* k_plane, const void* v_plane, long long page_stride, const int* positions,
     const int* token_slot, const int* block_table, int max_pages, int page_size, int dtype, int tokens,
     int q_heads, int kv_heads, int dk, int dv, float scale, float softcap, int chunk, int window, int sink,
-    const float* slopes, const float* sink_logit, const float* dist_bias, int dist_len, int v_row, const void* gate, int gate_stride, int gate_per_head, void* out, cudaStream_t stream) {
+    const float* slopes, const float* sink_logit, const float* dist_bias, int dist_len, int v_row, const void* gate, int gate_stride, int gate_per_head,
+    int maps, float lambda, float diff_eps, float diff_scale, void* out, cudaStream_t stream) {
     if (v_row <= 0) v_row = dv;
+    TLLM_REQUIRE(maps == 1 || (maps == 2 && diff_eps > 0.0f), "attention_biased: %d maps", maps);
+    const DiffMod diff{lambda, diff_eps, diff_scale};
     TLLM_REQUIRE(dist_bias == nullptr || dist_len > 0, "attention_biased: an empty table of biases");
     TLLM_REQUIRE(v_row >= dv, "attention_biased: values of width %d in rows of %d", dv, v_row);
     TLLM_REQUIRE(tokens >= 0 && q_heads > 0 && kv_heads > 0 && q_heads % kv_heads == 0,
@@ -1061,20 +1215,22 @@ int tllm_attention_biased_general(
     TLLM_REQUIRE(chunk >= 0 && window >= 0 && softcap >= 0.0f, "attention_biased: negative constant");
     if (tokens == 0) return 0;
     const ScoreMod mod{scale, softcap, chunk, window, sink ? 1 : 0, dist_bias, dist_len, gate_per_head ? 1 : 0};
-    if (dtype == kBF16)
-        return launch_general<bf16>(q, k_plane, v_plane, page_stride, positions, token_slot, block_table, max_pages,
-                                    page_size, tokens, q_heads, kv_heads, dk, dv, mod, slopes, sink_logit, v_row, gate, gate_stride, out, stream);
-    if (dtype == kF32)
-        return launch_general<float>(q, k_plane, v_plane, page_stride, positions, token_slot, block_table, max_pages,
-                                     page_size, tokens, q_heads, kv_heads, dk, dv, mod, slopes, sink_logit, v_row, gate, gate_stride, out, stream);
+#define GEN(T, M) launch_general<T, M>(q, k_plane, v_plane, page_stride, positions, token_slot, block_table, max_pages, page_size, \
+                                       tokens, q_heads, kv_heads, dk, dv, mod, diff, slopes, sink_logit, v_row, gate, gate_stride, out, stream)
+    if (dtype == kBF16) return maps == 2 ? GEN(bf16, 2) : GEN(bf16, 1);
+    if (dtype == kF32) return maps == 2 ? GEN(float, 2) : GEN(float, 1);
+#undef GEN
     TLLM_REQUIRE(false, "attention_biased: unknown dtype %d", dtype);
 }
 
-// Whether the two bfloat16 kernels below take these sizes (else the general kernel serves).
-int tllm_attention_biased_fast_ok(int q_heads, int kv_heads, int dk, int dv) {
-    return q_heads > 0 && kv_heads > 0 && q_heads % kv_heads == 0 && biased_sub_groups(q_heads / kv_heads) > 0 &&
-           kv_heads * biased_sub_groups(q_heads / kv_heads) <= 65535 &&
+// Whether the two bfloat16 kernels below take these sizes (else the general kernel serves).  dk: width of one map's key.
+int tllm_attention_maps_fast_ok(int q_heads, int kv_heads, int dk, int dv, int maps) {
+    return q_heads > 0 && kv_heads > 0 && q_heads % kv_heads == 0 && biased_sub_groups(q_heads / kv_heads, maps) > 0 &&
+           kv_heads * biased_sub_groups(q_heads / kv_heads, maps) <= 65535 &&
            dk % 8 == 0 && dv % 8 == 0 && dk > 0 && dv > 0 && dk <= 128 && dv <= 128;
+}
+int tllm_attention_biased_fast_ok(int q_heads, int kv_heads, int dk, int dv) {
+    return tllm_attention_maps_fast_ok(q_heads, kv_heads, dk, dv, 1);
 }
 
 // seg_info: int[segments][4] = slot, first row, length, position of the first row.
@@ -1083,46 +1239,56 @@ int tllm_attention_biased_prefill(
     const void* q, const void* k_plane, const void* v_plane, long long page_stride, const int* seg_info,
     const int* tiles, int n_tiles, const int* block_table, int max_pages, int page_size, int q_heads,
     int kv_heads, int dk, int dv, float scale, float softcap, int chunk, int window, int sink,
-    const float* slopes, const float* sink_logit, const float* dist_bias, int dist_len, int v_row, const void* gate, int gate_stride, int gate_per_head, void* out, cudaStream_t stream) {
+    const float* slopes, const float* sink_logit, const float* dist_bias, int dist_len, int v_row, const void* gate, int gate_stride, int gate_per_head,
+    int maps, float lambda, float diff_eps, float diff_scale, void* out, cudaStream_t stream) {
     if (v_row <= 0) v_row = dv;
+    TLLM_REQUIRE(maps == 1 || (maps == 2 && diff_eps > 0.0f), "attention_biased_prefill: %d maps", maps);
+    const DiffMod diff{lambda, diff_eps, diff_scale};
     TLLM_REQUIRE(dist_bias == nullptr || dist_len > 0, "attention_biased_prefill: an empty table of biases");
     TLLM_REQUIRE(v_row >= dv && v_row % 8 == 0, "attention_biased_prefill: values of width %d in rows of %d", dv, v_row);
-    TLLM_REQUIRE(tllm_attention_biased_fast_ok(q_heads, kv_heads, dk, dv), "attention_biased_prefill: sizes %d/%d heads, widths %d/%d", q_heads, kv_heads, dk, dv);
+    TLLM_REQUIRE(tllm_attention_maps_fast_ok(q_heads, kv_heads, dk, dv, maps), "attention_biased_prefill: sizes %d/%d heads, widths %d/%d", q_heads, kv_heads, dk, dv);
     TLLM_REQUIRE(page_size > 0 && max_pages > 0 && n_tiles >= 0 && q_heads <= 65535, "attention_biased_prefill: bad geometry");
     TLLM_REQUIRE(chunk >= 0 && window >= 0 && softcap >= 0.0f, "attention_biased_prefill: negative constant");
     TLLM_REQUIRE(gate == nullptr || gate_per_head || gate_stride % 2 == 0, "attention_biased_prefill: odd gate stride");
     if (n_tiles == 0) return 0;
     const ScoreMod mod{scale, softcap, chunk, window, sink ? 1 : 0, dist_bias, dist_len, gate_per_head ? 1 : 0};
-#define PF(A, B) launch_biased_prefill<A, B>(q, k_plane, v_plane, page_stride, seg_info, tiles, n_tiles, block_table, max_pages, \
-                                             page_size, q_heads, kv_heads, dk, dv, mod, slopes, sink_logit, v_row, gate, gate_stride, out, stream)
+#define PF_M(A, B, M) launch_biased_prefill<A, B, M>(q, k_plane, v_plane, page_stride, seg_info, tiles, n_tiles, block_table, max_pages, \
+                                             page_size, q_heads, kv_heads, dk, dv, mod, diff, slopes, sink_logit, v_row, gate, gate_stride, out, stream)
+#define PF(A, B) (maps == 2 ? PF_M(A, B, 2) : PF_M(A, B, 1))
     if (dk <= 64) return dv <= 64 ? PF(64, 64) : PF(64, 128);
     return dv <= 64 ? PF(128, 64) : PF(128, 128);
 #undef PF
+#undef PF_M
 }
 
 // rows: indices of the one-token rows (null: rows 0 .. n_rows - 1).  splits: runs of keys per (row,
-// key/value head), each a block; with more than one, `part` holds n_rows * q_heads * splits * (dv + 2) floats.
+// key/value head), each a block; with more than one, `part` holds n_rows * q_heads * maps * splits * (dv + 2) floats.
 int tllm_attention_biased_decode(
     const void* q, const void* k_plane, const void* v_plane, long long page_stride, const int* positions,
     const int* token_slot, const int* rows, int n_rows, const int* block_table, int max_pages, int page_size,
     int q_heads, int kv_heads, int dk, int dv, float scale, float softcap, int chunk, int window, int sink,
     const float* slopes, const float* sink_logit, const float* dist_bias, int dist_len, int v_row, const void* gate,
-    int gate_stride, int gate_per_head, int splits, float* part, void* out, cudaStream_t stream) {
+    int gate_stride, int gate_per_head, int maps, float lambda, float diff_eps, float diff_scale, int splits, float* part,
+    void* out, cudaStream_t stream) {
     if (v_row <= 0) v_row = dv;
+    TLLM_REQUIRE(maps == 1 || (maps == 2 && diff_eps > 0.0f), "attention_biased_decode: %d maps", maps);
+    const DiffMod diff{lambda, diff_eps, diff_scale};
     TLLM_REQUIRE(dist_bias == nullptr || dist_len > 0, "attention_biased_decode: an empty table of biases");
     TLLM_REQUIRE(v_row >= dv && v_row % 8 == 0, "attention_biased_decode: values of width %d in rows of %d", dv, v_row);
-    TLLM_REQUIRE(tllm_attention_biased_fast_ok(q_heads, kv_heads, dk, dv), "attention_biased_decode: sizes %d/%d heads, widths %d/%d", q_heads, kv_heads, dk, dv);
+    TLLM_REQUIRE(tllm_attention_maps_fast_ok(q_heads, kv_heads, dk, dv, maps), "attention_biased_decode: sizes %d/%d heads, widths %d/%d", q_heads, kv_heads, dk, dv);
     TLLM_REQUIRE(page_size > 0 && max_pages > 0 && n_rows >= 0 && kv_heads <= 65535, "attention_biased_decode: bad geometry");
     TLLM_REQUIRE(chunk >= 0 && window >= 0 && softcap >= 0.0f, "attention_biased_decode: negative constant");
     TLLM_REQUIRE(splits >= 1 && splits <= 64 && (splits == 1 || part != nullptr), "attention_biased_decode: %d runs of keys", splits);
     if (n_rows == 0) return 0;
     const ScoreMod mod{scale, softcap, chunk, window, sink ? 1 : 0, dist_bias, dist_len, gate_per_head ? 1 : 0};
-#define DEC(A, B) launch_biased_decode<A, B>(q, k_plane, v_plane, page_stride, positions, token_slot, rows, n_rows, block_table, \
-                                             max_pages, page_size, q_heads, kv_heads, dk, dv, mod, slopes, sink_logit, v_row, gate, gate_stride, \
+#define DEC_M(A, B, M) launch_biased_decode<A, B, M>(q, k_plane, v_plane, page_stride, positions, token_slot, rows, n_rows, block_table, \
+                                             max_pages, page_size, q_heads, kv_heads, dk, dv, mod, diff, slopes, sink_logit, v_row, gate, gate_stride, \
                                              splits, part, out, stream)
+#define DEC(A, B) (maps == 2 ? DEC_M(A, B, 2) : DEC_M(A, B, 1))
     if (dk <= 64) return dv <= 64 ? DEC(64, 64) : DEC(64, 128);
     return dv <= 64 ? DEC(128, 64) : DEC(128, 128);
 #undef DEC
+#undef DEC_M
 }
 
 }  // extern "C"

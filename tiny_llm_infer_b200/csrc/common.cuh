@@ -23,7 +23,14 @@ template <> __device__ __forceinline__ float from_f32<float>(float v) { return v
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
 
 // Activation of the gate in a gated feed-forward unit, act(gate) * up, by code.
-enum GateAct : int { kActSilu = 0, kActGeluTanh = 1, kActGeluErf = 2, kActRelu2 = 3 };
+// kActClampedSwish belongs to gated units only: it bounds gate and up before they meet (`gated_unit`).
+// kActTanh belongs to plain products only.
+enum GateAct : int { kActSilu = 0, kActGeluTanh = 1, kActGeluErf = 2, kActRelu2 = 3, kActClampedSwish = 4, kActTanh = 5 };
+
+// Constants of a gated unit whose activation has some (kActClampedSwish).
+struct GateConst {
+    float limit, slope;
+};
 
 __device__ __forceinline__ float gate_act(float g, int act) {
     if (act == kActGeluTanh)   // 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3)))
@@ -34,7 +41,19 @@ __device__ __forceinline__ float gate_act(float g, int act) {
         const float r = fmaxf(g, 0.0f);
         return r * r;
     }
+    if (act == kActTanh) return tanhf(g);
     return g / (1.0f + expf(-g));
+}
+
+// A gated unit's output from its gate and up sums: act(gate) * up, or, clamped, g sigmoid(slope g) (u + 1) with
+// g = min(gate, limit) and u = up held within -limit .. limit.
+__device__ __forceinline__ float gated_unit(float g, float u, int act, const GateConst& c) {
+    if (act == kActClampedSwish) {
+        g = fminf(g, c.limit);
+        u = fminf(fmaxf(u, -c.limit), c.limit);
+        return g / (1.0f + expf(-c.slope * g)) * (u + 1.0f);
+    }
+    return gate_act(g, act) * u;
 }
 
 __device__ __forceinline__ float warp_sum(float v) {

@@ -13,7 +13,7 @@
 //                  the others, so a thread keeps a slice of one column in registers (the dk rows are dealt
 //                  to R neighbouring lanes, which add their partial dot products with shuffles) and walks
 //                  the portion's tokens, which come through two stages of shared memory sixteen at a time
-//                  (cp.async: the next sixteen are on their way while these are walked).
+//                  (cp.async: the next sixteen are on their way while these are walked; eight for the widest keys).
 //   delta_finish   one block per token: o divided by its root mean square per head, times a weight, times
 //                  sigmoid(gate); the block of a portion's last token also moves the convolution's
 //                  window of the request's state on.
@@ -26,7 +26,9 @@
 namespace tllm {
 
 constexpr int kScanMaxPer = 16;     // rows of a column that one thread keeps
-constexpr int kScanChunk = 16;      // tokens staged at a time
+
+// Tokens staged at a time: sixteen, eight where 32 lanes share a column (the widest keys), whose rows would not fit.
+__host__ __device__ constexpr int scan_chunk(int lanes) { return lanes >= 32 ? 8 : 16; }
 
 static inline int delta_lanes(int dk) {
     int r = 4;
@@ -251,11 +253,12 @@ __device__ __forceinline__ void cp_async_f32x4(float* dst, const float* src) {
 // A lane r of a column keeps the rows i = r * per + il, il < per, as PER registers; in shared memory a token's
 // k (and q, g) row is laid out [R][PER + 4]: a lane's rows are neighbours, so it reads them four at a time, and
 // the four floats between the lanes' runs keep those reads off each other's banks.
-template <int R, int PER>
+template <int R, int PER, int VECS>
 struct ScanLayout {
-    static constexpr int kRow = R * (PER + 4);                               // floats of one token's k (or q, g) row
-    __host__ __device__ static constexpr int stage_floats(int cols) {       // k, q, g, the value columns, the betas, the keeps
-        return (kScanChunk * (3 * kRow + cols + 2) + 3) / 4 * 4;
+    static constexpr int kChunk = scan_chunk(R);
+    static constexpr int kRow = R * (PER + 4);                               // floats of one token's k (or q, g, e) row
+    __host__ __device__ static constexpr int stage_floats(int cols) {       // k, q, g (, e), the value columns, the betas, the keeps
+        return (kChunk * (VECS * kRow + cols + 2) + 3) / 4 * 4;
     }
 };
 
@@ -271,8 +274,11 @@ struct ScanLayout {
 // normaliser (the prepare kernel feeds it ones), whose read-out leaves as max(|n . q|, exp(-m')) + floor_eps in
 // `den` while the other columns go to o_raw [., heads, dv - 1].  kScanHeadDecay: kScanPlain with one decay per
 // (token, head) for all rows of S and a write strength likewise, S <- a S + k (w v)^T; the decays come in `beta`
-// [., heads], the strengths in `fgate` [., heads], and `decay` is not read.
-enum ScanMode : int { kScanDelta = 0, kScanPlain = 1, kScanMemory = 2, kScanHeadDecay = 3 };
+// [., heads], the strengths in `fgate` [., heads], and `decay` is not read.  kScanErase: a delta rule whose removal has
+// a rate per key channel and reads the state before its decay, S <- g S - e (k^T S)^T + k v^T with k the unit key and
+// e = rate * k in `erase` (v comes already multiplied by the key's length); no beta.
+enum ScanMode : int { kScanDelta = 0, kScanPlain = 1, kScanMemory = 2, kScanHeadDecay = 3, kScanErase = 4 };
+__host__ __device__ constexpr int scan_vecs(int mode) { return mode == kScanErase ? 4 : 3; }
 
 template <int R, int PER, int MODE>
 __global__ void __launch_bounds__(256, 2)
@@ -280,9 +286,11 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
                   const float* qn, const float* kn, const float* vv, const float* decay,
                   const float* beta, float* state, long long state_stride, int heads,
                   int kv_heads, int dk, int dv, int cols, int vec, float* o_raw,
-                  const float* fgate, long long aux_off, float floor_eps, float* den) {
+                  const float* fgate, const float* erase, long long aux_off, float floor_eps, float* den) {
     extern __shared__ __align__(16) float sm[];
-    using L = ScanLayout<R, PER>;
+    using L = ScanLayout<R, PER, scan_vecs(MODE)>;
+    constexpr int kScanChunk = L::kChunk;
+    constexpr bool kDecayRows = MODE == kScanDelta || MODE == kScanPlain || MODE == kScanErase;
     constexpr int kLane = PER + 4;
     TLLM_PDL_ENTER();
     const int seg = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * cols;
@@ -311,7 +319,8 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
         float* k_s = sm + st * stage_floats;
         float* q_s = k_s + kScanChunk * L::kRow;
         float* g_s = q_s + kScanChunk * L::kRow;
-        float* v_s = g_s + kScanChunk * L::kRow;
+        float* e_s = g_s + kScanChunk * L::kRow;
+        float* v_s = e_s + (MODE == kScanErase ? kScanChunk * L::kRow : 0);
         float* b_s = v_s + kScanChunk * cols;
         float* f_s = b_s + kScanChunk;
         if (vec) {                                    // dk and per multiples of four: four rows of one lane at a time
@@ -322,7 +331,8 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
                 const size_t row = (size_t)(start + c0 + tt);
                 cp_async_f32x4(k_s + at, kn + (row * kv_heads + kvh) * dk + e);
                 cp_async_f32x4(q_s + at, qn + (row * kv_heads + kvh) * dk + e);
-                if (MODE == kScanDelta || MODE == kScanPlain) cp_async_f32x4(g_s + at, decay + (row * heads + head) * dk + e);
+                if (kDecayRows) cp_async_f32x4(g_s + at, decay + (row * heads + head) * dk + e);
+                if (MODE == kScanErase) cp_async_f32x4(e_s + at, erase + (row * heads + head) * dk + e);
             }
         } else {
             for (int i = threadIdx.x; i < n * dk; i += blockDim.x) {
@@ -331,7 +341,8 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
                 const size_t row = (size_t)(start + c0 + tt);
                 cp_async_f32(k_s + at, kn + (row * kv_heads + kvh) * dk + e, true);
                 cp_async_f32(q_s + at, qn + (row * kv_heads + kvh) * dk + e, true);
-                if (MODE == kScanDelta || MODE == kScanPlain) cp_async_f32(g_s + at, decay + (row * heads + head) * dk + e, true);
+                if (kDecayRows) cp_async_f32(g_s + at, decay + (row * heads + head) * dk + e, true);
+                if (MODE == kScanErase) cp_async_f32(e_s + at, erase + (row * heads + head) * dk + e, true);
             }
         }
         for (int i = threadIdx.x; i < n * cols; i += blockDim.x) {
@@ -374,7 +385,8 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
         const float* k_s = sm + stage * stage_floats;
         const float* q_s = k_s + kScanChunk * L::kRow;
         const float* g_s = q_s + kScanChunk * L::kRow;
-        const float* v_s = g_s + kScanChunk * L::kRow;
+        const float* e_s = g_s + kScanChunk * L::kRow;
+        const float* v_s = e_s + (MODE == kScanErase ? kScanChunk * L::kRow : 0);
         const float* b_s = v_s + kScanChunk * cols;
         const float* f_s = b_s + kScanChunk;
         // every thread walks the tokens (the shuffles want whole warps); one without a column carries zeros
@@ -384,6 +396,7 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
             const float4* kr = reinterpret_cast<const float4*>(k_s + tt * L::kRow + r * kLane);
             const float4* qr = reinterpret_cast<const float4*>(q_s + tt * L::kRow + r * kLane);
             const float4* gr = reinterpret_cast<const float4*>(g_s + tt * L::kRow + r * kLane);
+            const float4* er = reinterpret_cast<const float4*>(e_s + tt * L::kRow + r * kLane);
             float2 kk[PER / 2];
             float2 dot_a = make_float2(0.0f, 0.0f), dot_b = dot_a;
             float write = 1.0f;
@@ -406,6 +419,10 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
                 const float4 k4 = kr[il >> 2];
                 kk[il >> 1] = make_float2(k4.x, k4.y);
                 kk[(il >> 1) + 1] = make_float2(k4.z, k4.w);
+                if (MODE == kScanErase) {                 // the removal reads the state before its decay
+                    dot_a = __ffma2_rn(S2[il >> 1], kk[il >> 1], dot_a);
+                    dot_b = __ffma2_rn(S2[(il >> 1) + 1], kk[(il >> 1) + 1], dot_b);
+                }
                 if (MODE == kScanMemory || MODE == kScanHeadDecay) {
                     S2[il >> 1] = __fmul2_rn(S2[il >> 1], keep2);
                     S2[(il >> 1) + 1] = __fmul2_rn(S2[(il >> 1) + 1], keep2);
@@ -420,7 +437,13 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
                 }
             }
             float u;
-            if (MODE == kScanDelta) {
+            float2 gone = make_float2(0.0f, 0.0f);
+            if (MODE == kScanErase) {
+                const float2 dsum = __fadd2_rn(dot_a, dot_b);
+                const float dot = -lanes_sum<R>(dsum.x + dsum.y);
+                gone = make_float2(dot, dot);
+                u = v_s[tt * cols + jl];
+            } else if (MODE == kScanDelta) {
                 const float2 dsum = __fadd2_rn(dot_a, dot_b);
                 const float dot = lanes_sum<R>(dsum.x + dsum.y);
                 u = b_s[tt] * (v_s[tt * cols + jl] - dot);
@@ -432,6 +455,11 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
 #pragma unroll
             for (int il = 0; il < PER; il += 4) {
                 const float4 q4 = qr[il >> 2];
+                if (MODE == kScanErase) {
+                    const float4 e4 = er[il >> 2];
+                    S2[il >> 1] = __ffma2_rn(make_float2(e4.x, e4.y), gone, S2[il >> 1]);
+                    S2[(il >> 1) + 1] = __ffma2_rn(make_float2(e4.z, e4.w), gone, S2[(il >> 1) + 1]);
+                }
                 S2[il >> 1] = __ffma2_rn(kk[il >> 1], u2, S2[il >> 1]);
                 S2[(il >> 1) + 1] = __ffma2_rn(kk[(il >> 1) + 1], u2, S2[(il >> 1) + 1]);
                 o_a = __ffma2_rn(S2[il >> 1], make_float2(q4.x, q4.y), o_a);
@@ -646,6 +674,97 @@ __global__ void linear_prepare_kernel(const T* proj, int ld, const float* z, int
     }
 }
 
+// ---------------------------------------------------------------- inputs of the delta rule with a removal rate per channel
+// proj[t] = r | k | v | gate | a in the storage type (heads x dk, heads x dk, heads x dv, heads x dv, heads x dk), z
+// [T, heads * dk] float32 the decay's logits.  Per head, with n = sqrt(sum(k^2) + unit_eps):
+//   qn = r,  kn = k / n,  vv = v n  (so that kn vv^T = k v^T),  decay = exp(-rate sigmoid(z + z_bias)),
+//   erase = sigmoid(a + a_bias) kn.
+// One warp per head and token, all float32.
+template <typename T>
+__global__ void erase_prepare_kernel(const T* proj, int ld, int a_col, const float* z, int ldz, const float* __restrict__ z_bias,
+                                     const float* __restrict__ a_bias, float rate, const int* __restrict__ token_slot,
+                                     int heads, int dk, int dv, float unit_eps, float* qn, float* kn, float* vv, float* decay,
+                                     float* erase) {
+    TLLM_PDL_ENTER();
+    const int t = blockIdx.x;
+    if (token_slot[t] < 0) return;
+    const T* row = proj + (size_t)t * ld;
+    const int qk = heads * dk, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    for (int h = blockIdx.y * warps + (threadIdx.x >> 5); h < heads; h += gridDim.y * warps) {
+        const T* k = row + qk + (size_t)h * dk;
+        float sum = 0.0f;
+        for (int e = lane; e < dk; e += 32) { const float x = to_f32<T>(k[e]); sum += x * x; }
+        const float n = sqrtf(warp_sum(sum) + unit_eps), inv = 1.0f / n;
+        for (int e = lane; e < dk; e += 32) {
+            const int c = h * dk + e;
+            const size_t at = (size_t)t * qk + c;
+            const float u = to_f32<T>(k[e]) * inv;
+            qn[at] = to_f32<T>(row[c]);
+            kn[at] = u;
+            decay[at] = expf(-rate / (1.0f + expf(-(z[(size_t)t * ldz + c] + z_bias[c]))));
+            erase[at] = u / (1.0f + expf(-(to_f32<T>(row[a_col + c]) + a_bias[c])));
+        }
+        for (int e = lane; e < dv; e += 32) vv[((size_t)t * heads + h) * dv + e] = to_f32<T>(row[2 * qk + h * dv + e]) * n;
+    }
+}
+
+// The same with eight elements per lane and access: a group of GS lanes (a power of two, dk <= 8 GS) holds a head, so a
+// warp takes 32 / GS heads at once (dk and dv multiples of eight, everything on 16-byte boundaries).
+template <typename T, int GS>
+__global__ void erase_prepare_vec_kernel(const T* proj, int ld, int a_col, const float* z, int ldz, const float* __restrict__ z_bias,
+                                         const float* __restrict__ a_bias, float rate, const int* __restrict__ token_slot,
+                                         int heads, int dk, int dv, float unit_eps, float* qn, float* kn, float* vv,
+                                         float* decay, float* erase) {
+    TLLM_PDL_ENTER();
+    const int t = blockIdx.x;
+    if (token_slot[t] < 0) return;
+    constexpr int kPerWarp = 32 / GS;
+    const T* row = proj + (size_t)t * ld;
+    const int qk = heads * dk, lane = threadIdx.x & 31, grp = lane / GS, e0 = (lane % GS) * 8;
+    const int per_block = (blockDim.x >> 5) * kPerWarp;
+    for (int base = blockIdx.y * per_block + (threadIdx.x >> 5) * kPerWarp; base < heads; base += gridDim.y * per_block) {
+        const int h = base + grp;                                   // every lane takes part in the exchange
+        const bool live = h < heads && e0 < dk;
+        const int c = h * dk + e0;
+        const size_t at = (size_t)t * qk + c;
+        float k[8] = {0, 0, 0, 0, 0, 0, 0, 0}, r[8], a[8], zz[8], zb[8], ab[8];
+        if (live) {
+            Ld8<T>::load(row + qk + c, k);
+            Ld8<T>::load(row + c, r);
+            Ld8<T>::load(row + a_col + c, a);
+            Ld8<float>::load(z + (size_t)t * ldz + c, zz);
+            Ld8<float>::load(z_bias + c, zb);
+            Ld8<float>::load(a_bias + c, ab);
+        }
+        float sum = 0.0f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum += k[e] * k[e];
+#pragma unroll
+        for (int o = GS / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+        const float n = sqrtf(sum + unit_eps), inv = 1.0f / n;
+        if (live) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                k[e] *= inv;
+                zz[e] = expf(-rate / (1.0f + expf(-(zz[e] + zb[e]))));
+                a[e] = k[e] / (1.0f + expf(-(a[e] + ab[e])));
+            }
+            Ld8<float>::store(qn + at, r);
+            Ld8<float>::store(kn + at, k);
+            Ld8<float>::store(decay + at, zz);
+            Ld8<float>::store(erase + at, a);
+        }
+        if (h < heads)
+            for (int e = e0; e < dv; e += GS * 8) {
+                float v[8];
+                Ld8<T>::load(row + 2 * qk + h * dv + e, v);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) v[i] *= n;
+                Ld8<float>::store(vv + ((size_t)t * heads + h) * dv + e, v);
+            }
+    }
+}
+
 }  // namespace tllm
 
 using namespace tllm;
@@ -672,6 +791,49 @@ int tllm_linear_prepare(const void* proj, int ld, int dtype, const float* z, int
                    z_bias, kind, p0, token_slot, heads, dk, dv, q_scale, qn, kn, vv, decay, wgate, fgate);
     else TLLM_REQUIRE(false, "linear_prepare: unknown dtype %d", dtype);
     return finish_launch("linear_prepare");
+}
+
+// See erase_prepare_kernel.  a_col: column of the removal rates' logits in a row of proj.
+int tllm_erase_prepare(const void* proj, int ld, int dtype, int a_col, const float* z, int ldz, const float* z_bias,
+                       const float* a_bias, float rate, const int* token_slot, int heads, int dk, int dv, float unit_eps,
+                       float* qn, float* kn, float* vv, float* decay, float* erase, int n_rows, cudaStream_t stream) {
+    TLLM_REQUIRE(n_rows >= 0 && heads > 0 && dk > 0 && dv > 0 && unit_eps > 0.0f, "erase_prepare: bad sizes");
+    TLLM_REQUIRE(a_col >= heads * (2 * dk + dv) && ld >= a_col + heads * dk && ldz >= heads * dk, "erase_prepare: rows too short");
+    TLLM_REQUIRE(dtype == kBF16 || dtype == kF32, "erase_prepare: unknown dtype %d", dtype);
+    if (n_rows == 0) return 0;
+    const auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; };
+    const bool vec = dk % 8 == 0 && dv % 8 == 0 && dk <= 256 && ld % 8 == 0 && a_col % 8 == 0 && ldz % 4 == 0 && al(proj) && al(z) &&
+                     al(z_bias) && al(a_bias) && al(qn) && al(kn) && al(vv) && al(decay) && al(erase);
+    int gs = 1;
+    while (gs * 8 < dk) gs *= 2;
+    const int per_warp = vec ? 32 / gs : 1;
+    // blocks per token: a warp's heads each where few rows leave the GPU empty
+    const int sms = sm_count_cached() > 0 ? sm_count_cached() : 148;
+    int warps = 8, split = 1;
+    while (warps > 1 && (warps / 2) * per_warp >= heads) warps /= 2;
+    while (split * warps * per_warp < heads && (long long)n_rows * split < 2LL * sms) split *= 2;
+    while (warps > 2 && split * 2 <= 64 && (long long)n_rows * split * 2 <= 2LL * sms) { warps /= 2; split *= 2; }
+    const dim3 grid(n_rows, split), block(warps * 32);
+#define EP(T) launch_pdl(kPdlOther, erase_prepare_kernel<T>, grid, block, 0, stream, (const T*)proj, ld, a_col, z, ldz, z_bias, a_bias, \
+                         rate, token_slot, heads, dk, dv, unit_eps, qn, kn, vv, decay, erase)
+#define EPV(T, G) launch_pdl(kPdlOther, erase_prepare_vec_kernel<T, G>, grid, block, 0, stream, (const T*)proj, ld, a_col, z, ldz, z_bias, \
+                             a_bias, rate, token_slot, heads, dk, dv, unit_eps, qn, kn, vv, decay, erase)
+#define EPG(T)                             \
+    do {                                   \
+        if (!vec) EP(T);                   \
+        else if (gs == 1) EPV(T, 1);       \
+        else if (gs == 2) EPV(T, 2);       \
+        else if (gs == 4) EPV(T, 4);       \
+        else if (gs == 8) EPV(T, 8);       \
+        else if (gs == 16) EPV(T, 16);     \
+        else EPV(T, 32);                   \
+    } while (0)
+    if (dtype == kBF16) EPG(bf16);
+    else EPG(float);
+#undef EPG
+#undef EPV
+#undef EP
+    return finish_launch("erase_prepare");
 }
 
 // Lanes that share a column of the state for keys of width dk (the state's layout depends on it).
@@ -751,14 +913,15 @@ int tllm_delta_prepare(const void* proj, int ld, int dtype, const void* conv_w, 
 int tllm_delta_scan(const int* seg_info, int segments, const int* token_slot, const float* qn, const float* kn,
                     const float* vv, const float* decay, const float* beta, float* state, long long state_stride,
                     int heads, int kv_heads, int dk, int dv, float* o_raw, int mode, const float* fgate,
-                    long long aux_off, float floor_eps, float* den, cudaStream_t stream) {
+                    const float* erase, long long aux_off, float floor_eps, float* den, cudaStream_t stream) {
     TLLM_REQUIRE(segments >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dk > 0 && dv > 0,
                  "delta_scan: bad sizes");
-    TLLM_REQUIRE(mode == kScanDelta || mode == kScanPlain || mode == kScanMemory || mode == kScanHeadDecay,
+    TLLM_REQUIRE(mode == kScanDelta || mode == kScanPlain || mode == kScanMemory || mode == kScanHeadDecay || mode == kScanErase,
                  "delta_scan: unknown recurrence %d", mode);
     TLLM_REQUIRE(mode == kScanMemory ? (beta != nullptr && fgate != nullptr && den != nullptr && dv >= 2 && aux_off > 0)
                  : mode == kScanHeadDecay ? (beta != nullptr && fgate != nullptr) : decay != nullptr, "delta_scan: the recurrence lacks an operand");
     TLLM_REQUIRE(mode != kScanDelta || beta != nullptr, "delta_scan: the delta rule needs its betas");
+    TLLM_REQUIRE(mode != kScanErase || (erase != nullptr && kv_heads == heads), "delta_scan: a removal per channel needs its rates and a key per head");
     TLLM_REQUIRE(heads <= 65535, "delta_scan: %d heads", heads);
     if (segments == 0) return 0;
     const int r = delta_lanes(dk), per = (dk + r - 1) / r;
@@ -775,17 +938,19 @@ int tllm_delta_scan(const int* seg_info, int segments, const int* token_slot, co
     const int threads = cols * r;
     TLLM_REQUIRE(col_blocks <= 65535, "delta_scan: sizes %d x %d do not fit", dk, dv);
     const auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; };
-    const int vec = dk % 4 == 0 && per % 4 == 0 && aligned(qn) && aligned(kn) && (decay == nullptr || aligned(decay));
+    const int vec = dk % 4 == 0 && per % 4 == 0 && aligned(qn) && aligned(kn) && (decay == nullptr || aligned(decay)) &&
+                    (erase == nullptr || aligned(erase));
 #define SCAN(RR, PP)                                                                                             \
     do {                                                                                                         \
         if (mode == kScanDelta) SCAN_MODE(RR, PP, kScanDelta);                                                   \
         else if (mode == kScanPlain) SCAN_MODE(RR, PP, kScanPlain);                                              \
         else if (mode == kScanHeadDecay) SCAN_MODE(RR, PP, kScanHeadDecay);                                      \
+        else if (mode == kScanErase) SCAN_MODE(RR, PP, kScanErase);                                              \
         else SCAN_MODE(RR, PP, kScanMemory);                                                                     \
     } while (0)
 #define SCAN_MODE(RR, PP, MM)                                                                                           \
     do {                                                                                                         \
-        const size_t smem = ((size_t)2 * ScanLayout<RR, PP>::stage_floats(cols) + (size_t)kScanChunk * cols) * sizeof(float); \
+        const size_t smem = ((size_t)2 * ScanLayout<RR, PP, scan_vecs(MM)>::stage_floats(cols) + (size_t)scan_chunk(RR) * cols) * sizeof(float); \
         TLLM_REQUIRE(smem <= 200 * 1024, "delta_scan: sizes %d x %d do not fit", dk, dv);                         \
         static OncePerDevice configured;                                                                         \
         if (configured.first()) {                                                                                \
@@ -795,7 +960,7 @@ int tllm_delta_scan(const int* seg_info, int segments, const int* token_slot, co
         }                                                                                                        \
         launch_pdl(kPdlOther, delta_scan_kernel<RR, PP, MM>, dim3(segments, heads, col_blocks), dim3(threads), smem, stream, \
                    seg_info, token_slot, qn, kn, vv, decay, beta, state, state_stride, heads, kv_heads, dk, dv,  \
-                   cols, vec, o_raw, fgate, aux_off, floor_eps, den);                                            \
+                   cols, vec, o_raw, fgate, erase, aux_off, floor_eps, den);                                            \
     } while (0)
     if (r == 4 && per <= 4) SCAN(4, 4);
     else if (r == 4 && per <= 8) SCAN(4, 8);

@@ -511,12 +511,12 @@ __global__ void postnorm_add_rmsnorm_vec_kernel(float* h, const TD* delta, const
 }
 
 // ---------------------------------------------------------------- SwiGLU
-// out[t, i] = act(gate) * up in float32; act is silu(x) = x / (1 + exp(-x)) or the tanh form of
-// GELU (`gate_act` in common.cuh).  Stacked columns: gate at
+// out[t, i] = act(gate) * up in float32; act is silu(x) = x / (1 + exp(-x)), the tanh form of
+// GELU or the clamped swish (`gated_unit` in common.cuh).  Stacked columns: gate at
 // gu[t, i], up at gu[t, inter + i].  Interleaved by eight: columns come in groups of sixteen,
 // eight gates followed by their eight ups, so gate at gu[t, 16 (i / 8) + i % 8] and up 8 further.
 template <typename T>
-__global__ void swiglu_kernel(const T* gu, T* out, int inter, int interleaved, int act,
+__global__ void swiglu_kernel(const T* gu, T* out, int inter, int interleaved, int act, GateConst gc,
                               size_t total) {
     TLLM_PDL_ENTER();
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -526,12 +526,12 @@ __global__ void swiglu_kernel(const T* gu, T* out, int inter, int interleaved, i
         const size_t gi = interleaved ? 16 * (i >> 3) + (i & 7) : i, ui = interleaved ? gi + 8 : inter + i;
         const float g = to_f32<T>(gu[t * 2 * inter + gi]);
         const float u = to_f32<T>(gu[t * 2 * inter + ui]);
-        out[idx] = from_f32<T>(gate_act(g, act) * u);
+        out[idx] = from_f32<T>(gated_unit(g, u, act, gc));
     }
 }
 
 template <typename T>
-__global__ void swiglu_vec_kernel(const T* gu, T* out, int inter, int interleaved, int act,
+__global__ void swiglu_vec_kernel(const T* gu, T* out, int inter, int interleaved, int act, GateConst gc,
                                   size_t total_chunks) {
     TLLM_PDL_ENTER();
     const int per_row = inter >> 3;
@@ -543,7 +543,7 @@ __global__ void swiglu_vec_kernel(const T* gu, T* out, int inter, int interleave
         Vec8<T>::load(gu + t * 2 * inter + (interleaved ? c * 16 : c * 8), g);
         Vec8<T>::load(gu + t * 2 * inter + (interleaved ? c * 16 + 8 : inter + c * 8), u);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) g[e] = gate_act(g[e], act) * u[e];
+        for (int e = 0; e < 8; ++e) g[e] = gated_unit(g[e], u[e], act, gc);
         Vec8<T>::store(out + t * inter + c * 8, g);
     }
 }
@@ -1070,7 +1070,7 @@ int tllm_softcap(float* x, float cap, long long n, cudaStream_t stream) {
 // out = act(x), times table[ids[t], col0 + j] where a table is given (x and out [tokens, width]).
 int tllm_activation(const void* x, void* out, int dtype, int act, int tokens, int width, const int* ids,
                     const void* table, int ldt, int col0, int vocab, cudaStream_t stream) {
-    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh || act == kActGeluErf || act == kActRelu2, "activation: unknown activation %d", act);
+    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh || act == kActGeluErf || act == kActRelu2 || act == kActTanh, "activation: unknown activation %d", act);
     TLLM_REQUIRE(tokens >= 0 && width > 0, "activation: bad sizes");
     TLLM_REQUIRE(table == nullptr || (ids != nullptr && col0 >= 0 && col0 + width <= ldt && vocab > 0), "activation: bad table");
     const size_t total = (size_t)tokens * width;
@@ -1127,9 +1127,11 @@ int tllm_postnorm_add_rmsnorm(float* h, const void* delta, const void* post_gain
     TLLM_REQUIRE(false, "postnorm_add_rmsnorm: unknown dtype %d", act_dtype);
 }
 
+// limit, slope: constants of the clamped swish (not looked at by the others).
 int tllm_swiglu(const void* gate_up, void* out, int dtype, int tokens, int inter, int interleaved,
-                int act, cudaStream_t stream) {
-    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh, "swiglu: unknown activation %d", act);
+                int act, float limit, float slope, cudaStream_t stream) {
+    const GateConst gc{limit, slope};
+    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh || (act == kActClampedSwish && limit > 0.0f), "swiglu: unknown activation %d", act);
     TLLM_REQUIRE(tokens >= 0 && inter > 0, "swiglu: bad sizes");
     TLLM_REQUIRE(!interleaved || inter % 8 == 0, "swiglu: interleaved columns need a multiple of 8, not %d", inter);
     TLLM_REQUIRE(dtype == kBF16 || dtype == kF32, "swiglu: unknown dtype %d", dtype);
@@ -1140,15 +1142,15 @@ int tllm_swiglu(const void* gate_up, void* out, int dtype, int tokens, int inter
         const size_t chunks = total / 8;
         const int grid = grid_for(chunks, block);
         if (dtype == kBF16)
-            launch_pdl(kPdlSwiglu, swiglu_vec_kernel<bf16>, dim3(grid), dim3(block), 0, stream, (const bf16*)gate_up, (bf16*)out, inter, interleaved, act, chunks);
+            launch_pdl(kPdlSwiglu, swiglu_vec_kernel<bf16>, dim3(grid), dim3(block), 0, stream, (const bf16*)gate_up, (bf16*)out, inter, interleaved, act, gc, chunks);
         else
-            launch_pdl(kPdlSwiglu, swiglu_vec_kernel<float>, dim3(grid), dim3(block), 0, stream, (const float*)gate_up, (float*)out, inter, interleaved, act, chunks);
+            launch_pdl(kPdlSwiglu, swiglu_vec_kernel<float>, dim3(grid), dim3(block), 0, stream, (const float*)gate_up, (float*)out, inter, interleaved, act, gc, chunks);
     } else {
         const int grid = grid_for(total, block);
         if (dtype == kBF16)
-            launch_pdl(kPdlSwiglu, swiglu_kernel<bf16>, dim3(grid), dim3(block), 0, stream, (const bf16*)gate_up, (bf16*)out, inter, interleaved, act, total);
+            launch_pdl(kPdlSwiglu, swiglu_kernel<bf16>, dim3(grid), dim3(block), 0, stream, (const bf16*)gate_up, (bf16*)out, inter, interleaved, act, gc, total);
         else
-            launch_pdl(kPdlSwiglu, swiglu_kernel<float>, dim3(grid), dim3(block), 0, stream, (const float*)gate_up, (float*)out, inter, interleaved, act, total);
+            launch_pdl(kPdlSwiglu, swiglu_kernel<float>, dim3(grid), dim3(block), 0, stream, (const float*)gate_up, (float*)out, inter, interleaved, act, gc, total);
     }
     return finish_launch("swiglu");
 }

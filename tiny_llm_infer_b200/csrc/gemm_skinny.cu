@@ -57,7 +57,7 @@ struct SkinnyStage {
 // 78) and with them the third block per SM (the gate/up product of Qwen3-8B sizes: 42.5 us at two
 // blocks per SM, 35.1 at three, as the plain product of the same rows).
 template <int NT, typename TOut, bool SWIGLU, int ACT, bool UNARY>
-__device__ __noinline__ void skinny_epilogue(float (*red)[16][NT * 8 + 1], TOut* y, int M, int N, int r0) {
+__device__ __noinline__ void skinny_epilogue(float (*red)[16][NT * 8 + 1], TOut* y, int M, int N, int r0, GateConst gc) {
     constexpr int kRows = SWIGLU ? 8 : 16;                   // output columns of the block
     for (int idx = threadIdx.x; idx < kRows * NT * 8; idx += blockDim.x) {
         const int row = idx % kRows, tok = idx / kRows;
@@ -69,7 +69,7 @@ __device__ __noinline__ void skinny_epilogue(float (*red)[16][NT * 8 + 1], TOut*
                 float up = 0.0f;
 #pragma unroll
                 for (int ww = 0; ww < kSkinnyWarps; ++ww) up += red[ww][row + 8][tok];
-                s = gate_act(s, ACT) * up;
+                s = gated_unit(s, up, ACT, gc);
             } else if (UNARY) {                              // a plain product with an activation on every output
                 s = gate_act(s, ACT);
             }
@@ -85,7 +85,7 @@ __device__ __noinline__ void skinny_epilogue(float (*red)[16][NT * 8 + 1], TOut*
 // pattern and the registers are those of the plain product of the 2 N rows.
 template <int NT, typename TOut, bool SWIGLU, int STAGES, int ACT, bool UNARY>
 __global__ void __launch_bounds__(kSkinnyWarps * 32)
-skinny_gemm_kernel(const bf16* x, const bf16* __restrict__ w, TOut* y, int M, int N, int K) {
+skinny_gemm_kernel(const bf16* x, const bf16* __restrict__ w, TOut* y, int M, int N, int K, GateConst gc) {
     __shared__ float red[kSkinnyWarps][16][NT * 8 + 1];
     asm volatile("griddepcontrol.launch_dependents;\n" ::);
     const int r0 = blockIdx.x * (SWIGLU ? 8 : 16);
@@ -169,11 +169,12 @@ skinny_gemm_kernel(const bf16* x, const bf16* __restrict__ w, TOut* y, int M, in
         red[warp][rq + 8][nt * 8 + c * 2 + 1] = acc[nt][3];
     }
     __syncthreads();
-    skinny_epilogue<NT, TOut, SWIGLU, ACT, UNARY>(red, y, M, N, r0);
+    skinny_epilogue<NT, TOut, SWIGLU, ACT, UNARY>(red, y, M, N, r0, gc);
 }
 
 template <int NT, typename TOut, bool SWIGLU, int STAGES = 3, int ACT = kActSilu, bool UNARY = false>
-static int launch_skinny(const void* x, const void* w, void* y, int M, int N, int K, cudaStream_t stream) {
+static int launch_skinny(const void* x, const void* w, void* y, int M, int N, int K, cudaStream_t stream,
+                         GateConst gc = GateConst{0.0f, 0.0f}) {
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(SWIGLU ? (N + 7) / 8 : (N + 15) / 16);
     cfg.blockDim = dim3(kSkinnyWarps * 32);
@@ -185,7 +186,7 @@ static int launch_skinny(const void* x, const void* w, void* y, int M, int N, in
     cfg.attrs = attr;
     cfg.numAttrs = 1;
     cudaError_t e = cudaLaunchKernelEx(&cfg, skinny_gemm_kernel<NT, TOut, SWIGLU, STAGES, ACT, UNARY>, (const bf16*)x, (const bf16*)w,
-                                       (TOut*)y, M, N, K);
+                                       (TOut*)y, M, N, K, gc);
     if (e != cudaSuccess) {
         set_error("gemm_skinny: %s", cudaGetErrorString(e));
         return (int)e;
@@ -230,11 +231,11 @@ extern "C" int tllm_gemm_skinny(const void* x, const void* w, void* y, int out_d
     return launch_skinny<4, float, false>(x, w, y, M, N, K, stream);
 }
 
-// y[M, N] = act(x . gate^T) * (x . up^T), act silu or the tanh form of GELU, for w of 2 N rows, gate and up interleaved by eight
-// (eight gate rows, their eight up rows, ...), bfloat16 out, M <= 16.
+// y[M, N] = act(x . gate^T) * (x . up^T), act silu, the tanh form of GELU or the clamped swish (with its constants),
+// for w of 2 N rows, gate and up interleaved by eight (eight gate rows, their eight up rows, ...), bfloat16 out, M <= 16.
 extern "C" int tllm_gemm_skinny_swiglu(const void* x, const void* w, void* y, int M, int N, int K, int act,
-                                       cudaStream_t stream) {
-    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh, "gemm_skinny_swiglu: unknown activation %d", act);
+                                       float limit, float slope, cudaStream_t stream) {
+    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh || (act == kActClampedSwish && limit > 0.0f), "gemm_skinny_swiglu: unknown activation %d", act);
     TLLM_REQUIRE(M >= 0 && N > 0 && K > 0, "gemm_skinny_swiglu: bad sizes");
     TLLM_REQUIRE(M <= 16, "gemm_skinny_swiglu: %d rows exceed 16", M);
     TLLM_REQUIRE(N % 8 == 0, "gemm_skinny_swiglu: N = %d is no multiple of 8", N);
@@ -246,15 +247,20 @@ extern "C" int tllm_gemm_skinny_swiglu(const void* x, const void* w, void* y, in
         if (M <= 8) return launch_skinny<1, bf16, true, 3, kActGeluTanh>(x, w, y, M, N, K, stream);
         return launch_skinny<2, bf16, true, 3, kActGeluTanh>(x, w, y, M, N, K, stream);
     }
+    if (act == kActClampedSwish) {
+        const GateConst gc{limit, slope};
+        if (M <= 8) return launch_skinny<1, bf16, true, 3, kActClampedSwish>(x, w, y, M, N, K, stream, gc);
+        return launch_skinny<2, bf16, true, 3, kActClampedSwish>(x, w, y, M, N, K, stream, gc);
+    }
     if (M <= 8) return launch_skinny<1, bf16, true>(x, w, y, M, N, K, stream);
     return launch_skinny<2, bf16, true>(x, w, y, M, N, K, stream);
 }
 
-// y[M, N] = act(x . w^T) for at most 8 rows, bfloat16 out: the plain product with silu, the tanh GELU or the
-// exact GELU on every output, in the same kernel.
+// y[M, N] = act(x . w^T) for at most 8 rows, bfloat16 out: the plain product with silu, the tanh GELU, the
+// exact GELU, the squared ReLU or tanh on every output, in the same kernel.
 extern "C" int tllm_gemm_skinny_act(const void* x, const void* w, void* y, int M, int N, int K, int act,
                                     cudaStream_t stream) {
-    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh || act == kActGeluErf || act == kActRelu2, "gemm_skinny_act: unknown activation %d", act);
+    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh || act == kActGeluErf || act == kActRelu2 || act == kActTanh, "gemm_skinny_act: unknown activation %d", act);
     TLLM_REQUIRE(M >= 0 && N > 0 && K > 0, "gemm_skinny_act: bad sizes");
     TLLM_REQUIRE(M <= 8, "gemm_skinny_act: %d rows exceed 8", M);
     TLLM_REQUIRE(K % 8 == 0, "gemm_skinny_act: K = %d is no multiple of 8", K);
@@ -262,6 +268,7 @@ extern "C" int tllm_gemm_skinny_act(const void* x, const void* w, void* y, int M
                  "gemm_skinny_act: operands must be 16-byte aligned");
     if (M == 0) return 0;
     if (act == kActGeluErf) return launch_skinny<1, bf16, false, 3, kActGeluErf, true>(x, w, y, M, N, K, stream);
+    if (act == kActTanh) return launch_skinny<1, bf16, false, 3, kActTanh, true>(x, w, y, M, N, K, stream);
     if (act == kActRelu2) return launch_skinny<1, bf16, false, 3, kActRelu2, true>(x, w, y, M, N, K, stream);
     if (act == kActGeluTanh) return launch_skinny<1, bf16, false, 3, kActGeluTanh, true>(x, w, y, M, N, K, stream);
     return launch_skinny<1, bf16, false, 3, kActSilu, true>(x, w, y, M, N, K, stream);

@@ -49,6 +49,17 @@ __device__ __forceinline__ float fast_gate_act(float g) {
     return __fdividef(g, 1.0f + __expf(-g));
 }
 
+// A gated unit's output the same way (`gated_unit` in common.cuh).
+template <int ACT>
+__device__ __forceinline__ float fast_gated_unit(float g, float u, const GateConst& c) {
+    if (ACT == kActClampedSwish) {
+        g = fminf(g, c.limit);
+        u = fminf(fmaxf(u, -c.limit), c.limit);
+        return __fdividef(g, 1.0f + __expf(-c.slope * g)) * (u + 1.0f);
+    }
+    return fast_gate_act<ACT>(g) * u;
+}
+
 // An activation on every output of a plain product (ACT: a GateAct code, or kActNone for none): silu and the
 // tanh GELU as above, the exact GELU 0.5 g (1 + erf(g / sqrt 2)) with the library's erff.
 constexpr int kActNone = -1;
@@ -56,6 +67,7 @@ template <int ACT>
 __device__ __forceinline__ float unary_act(float g) {
     if (ACT == kActGeluErf) return 0.5f * g * (1.0f + erff(g * 0.7071067811865476f));
     if (ACT == kActNone) return g;
+    if (ACT == kActTanh) return tanhf(g);
     if (ACT == kActRelu2) { const float r = fmaxf(g, 0.0f); return r * r; }
     return fast_gate_act<ACT>(g);
 }
@@ -191,7 +203,7 @@ template <bool SWIGLU, int MT, int ACT>
 __global__ void __launch_bounds__(kGemmThreads)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                     bf16* __restrict__ y, int M, int N, int K, int half_n, int interleaved, int tiles_m,
-                    int tiles_n, int* __restrict__ error_word, const GroupedTiles grouped) {
+                    int tiles_n, int* __restrict__ error_word, const GroupedTiles grouped, const GateConst gc) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     __shared__ __align__(8) uint64_t full_bar[4], empty_bar[4], acc_full[2], acc_empty[2];
     __shared__ uint32_t tmem_base_slot;
@@ -348,8 +360,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
                             for (int i = 0; i < 16; ++i) {
                                 const int gi = 16 * (i >> 3) + (i & 7);
                                 const float g0 = __uint_as_float(r0[gi]), g1 = __uint_as_float(r1[gi]);
-                                v[32 * h + i] = fast_gate_act<ACT>(g0) * __uint_as_float(r0[gi + 8]);
-                                v[32 * h + 16 + i] = fast_gate_act<ACT>(g1) * __uint_as_float(r1[gi + 8]);
+                                v[32 * h + i] = fast_gated_unit<ACT>(g0, __uint_as_float(r0[gi + 8]), gc);
+                                v[32 * h + 16 + i] = fast_gated_unit<ACT>(g1, __uint_as_float(r1[gi + 8]), gc);
                             }
                         }
                     } else if (SWIGLU) {
@@ -362,7 +374,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
 #pragma unroll
                             for (int i = 0; i < 32; ++i) {
                                 const float g = __uint_as_float(gr[i]);
-                                v[32 * h + i] = fast_gate_act<ACT>(g) * __uint_as_float(ur[i]);
+                                v[32 * h + i] = fast_gated_unit<ACT>(g, __uint_as_float(ur[i]), gc);
                             }
                         }
                     } else {
@@ -460,7 +472,7 @@ template <bool SWIGLU, int MT, int ACT = (SWIGLU ? (int)kActSilu : kActNone)>
 static int launch_tcgen05(const CUtensorMap& mx, const CUtensorMap& mw, void* y, int M, int N, int K, int half_n,
                           int interleaved, int* error_word, cudaStream_t stream,
                           const GroupedTiles grouped = GroupedTiles{nullptr, nullptr, nullptr, nullptr, 0},
-                          int grouped_max_tiles = 0) {
+                          int grouped_max_tiles = 0, const GateConst gc = GateConst{0.0f, 0.0f}) {
     const size_t smem = (size_t)(MT == 1 ? 4 : 3) * (kBM * MT * kBK * 2 + kStageBBytes) + 1024 + 4 * 32 * (64 * 2 + 16);
     static OncePerDevice configured;
     if (configured.first()) {
@@ -476,7 +488,7 @@ static int launch_tcgen05(const CUtensorMap& mx, const CUtensorMap& mw, void* y,
     const int total = tiles_m * tiles_n;
     const int grid = total < sm_count() ? total : sm_count();
     gemm_tcgen05_kernel<SWIGLU, MT, ACT><<<grid, kGemmThreads, smem, stream>>>(mx, mw, (bf16*)y, M, N, K, half_n, interleaved,
-                                                                      tiles_m, tiles_n, error_word, grouped);
+                                                                      tiles_m, tiles_n, error_word, grouped, gc);
     return finish_launch("gemm_tcgen05");
 }
 
@@ -486,11 +498,12 @@ using namespace tllm;
 
 // y = x . w^T (y is [M, N]) or, with bit 1 of `swiglu`, y = silu(x . gate^T) * (x . up^T) (y is
 // [M, N / 2]) for w = [gate; up], or with bit 4 as well for gate and up rows interleaved by eight.
+// Bits 8 and up: the activation (GateAct); limit, slope: constants of the clamped swish.
 // Bit 2 keeps blocks of 128 rows.  x [M, K], w [N, K] bfloat16 row-major, K a multiple of 8,
 // operands 16-byte aligned.  `error_word` is a device int the kernel sets to a non-zero code if
 // one of its bounded waits ran out (the result is then invalid); the caller clears and reads it.
 extern "C" int tllm_gemm_tcgen05(const void* x, const void* w, void* y, int M, int N, int K, int swiglu,
-                                 int* error_word, cudaStream_t stream) {
+                                 float limit, float slope, int* error_word, cudaStream_t stream) {
     TLLM_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_tcgen05: bad sizes");
     TLLM_REQUIRE(K % 8 == 0, "gemm_tcgen05: K = %d is no multiple of 8", K);
     TLLM_REQUIRE(!(swiglu & 1) || N % 2 == 0, "gemm_tcgen05: SwiGLU needs an even number of weight rows");
@@ -513,10 +526,17 @@ extern "C" int tllm_gemm_tcgen05(const void* x, const void* w, void* y, int M, i
         if (act == kActGeluTanh) return UNARY(kActGeluTanh);
         if (act == kActSilu) return UNARY(kActSilu);
         if (act == kActRelu2) return UNARY(kActRelu2);
+        if (act == kActTanh) return UNARY(kActTanh);
 #undef UNARY
         TLLM_REQUIRE(false, "gemm_tcgen05: unknown activation %d", act);
     }
-    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh, "gemm_tcgen05: unknown activation %d", act);
+    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh || (act == kActClampedSwish && limit > 0.0f), "gemm_tcgen05: unknown activation %d", act);
+    if ((swiglu & 1) && act == kActClampedSwish) {
+        const GateConst gc{limit, slope};
+        const GroupedTiles plain{nullptr, nullptr, nullptr, nullptr, 0};
+        return tall ? launch_tcgen05<true, 2, kActClampedSwish>(mx, mw, y, M, N, K, N / 2, interleaved, error_word, stream, plain, 0, gc)
+                    : launch_tcgen05<true, 1, kActClampedSwish>(mx, mw, y, M, N, K, N / 2, interleaved, error_word, stream, plain, 0, gc);
+    }
     if ((swiglu & 1) && act == kActGeluTanh)
         return tall ? launch_tcgen05<true, 2, kActGeluTanh>(mx, mw, y, M, N, K, N / 2, interleaved, error_word, stream)
                     : launch_tcgen05<true, 1, kActGeluTanh>(mx, mw, y, M, N, K, N / 2, interleaved, error_word, stream);
@@ -532,7 +552,8 @@ extern "C" int tllm_gemm_tcgen05(const void* x, const void* w, void* y, int M, i
 // tllm_gemm_tcgen05 (bit 1 with bit 4: gate and up rows interleaved by eight, y is [rows, n / 2]).
 extern "C" int tllm_gemm_tcgen05_grouped(const void* x, const void* w, void* y, int rows, int n, int K, int experts,
                                          int flags, const int* tile_expert, const int* tile_row0, const int* n_tiles,
-                                         const int* offsets, int max_tiles, int* error_word, cudaStream_t stream) {
+                                         const int* offsets, int max_tiles, float limit, float slope, int* error_word,
+                                         cudaStream_t stream) {
     TLLM_REQUIRE(rows > 0 && n > 0 && K > 0 && experts > 0 && max_tiles > 0, "gemm_tcgen05_grouped: bad sizes");
     TLLM_REQUIRE(K % 8 == 0, "gemm_tcgen05_grouped: K = %d is no multiple of 8", K);
     const bool gated = flags & 1;
@@ -550,13 +571,17 @@ extern "C" int tllm_gemm_tcgen05_grouped(const void* x, const void* w, void* y, 
         TLLM_REQUIRE(!gated, "gemm_tcgen05_grouped: either a gated or a plain activation");
 #define UNARY(A) launch_tcgen05<false, 1, A>(mx, mw, y, rows, n, K, 0, 0, error_word, stream, grouped, max_tiles)
         if (act == kActRelu2) return UNARY(kActRelu2);
+        if (act == kActTanh) return UNARY(kActTanh);
         if (act == kActSilu) return UNARY(kActSilu);
         if (act == kActGeluTanh) return UNARY(kActGeluTanh);
         if (act == kActGeluErf) return UNARY(kActGeluErf);
 #undef UNARY
         TLLM_REQUIRE(false, "gemm_tcgen05_grouped: unknown activation %d", act);
     }
-    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh, "gemm_tcgen05_grouped: unknown activation %d", act);
+    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh || (act == kActClampedSwish && limit > 0.0f), "gemm_tcgen05_grouped: unknown activation %d", act);
+    if (gated && act == kActClampedSwish)
+        return launch_tcgen05<true, 1, kActClampedSwish>(mx, mw, y, rows, n, K, n / 2, 1, error_word, stream, grouped, max_tiles,
+                                                         GateConst{limit, slope});
     if (gated && act == kActGeluTanh)
         return launch_tcgen05<true, 1, kActGeluTanh>(mx, mw, y, rows, n, K, n / 2, 1, error_word, stream, grouped, max_tiles);
     if (gated) return launch_tcgen05<true, 1>(mx, mw, y, rows, n, K, n / 2, 1, error_word, stream, grouped, max_tiles);

@@ -67,9 +67,10 @@ __global__ void moe_route_kernel(const float* z, int tokens, int experts, int to
 // Routing over scores of all experts.  One warp per token, E <= 1024; shared memory per warp: E choice scores,
 // then one number per group.  score s = softmax(z) over all E (score_mode 1) or sigmoid(z) (0); choice = s +
 // correction (if given); a group's score is its largest choice; only experts of the `keep` best groups can be
-// chosen (lowest index first on ties, for groups and experts alike); weights are the scores s themselves.
-__global__ void moe_route_grouped_kernel(const float* z, int tokens, int experts, int top, int score_mode,
-                                         const float* __restrict__ correction, int groups, int keep,
+// chosen (lowest index first on ties, for groups and experts alike); weights are the scores s themselves, times
+// `scale`.  A row of z is `ldz` floats long (other outputs of the same product may follow the logits).
+__global__ void moe_route_grouped_kernel(const float* z, int ldz, int tokens, int experts, int top, int score_mode,
+                                         const float* __restrict__ correction, int groups, int keep, float scale,
                                          int* __restrict__ ids, float* __restrict__ weights) {
     extern __shared__ float route_smem[];
     TLLM_PDL_ENTER();
@@ -78,7 +79,7 @@ __global__ void moe_route_grouped_kernel(const float* z, int tokens, int experts
     if (warp >= tokens) return;
     float* choice = route_smem + (size_t)wib * (experts + groups);
     float* gscore = choice + experts;
-    const float* row = z + (size_t)warp * experts;
+    const float* row = z + (size_t)warp * ldz;
     float top_z = -INFINITY;
     for (int e = lane; e < experts; e += 32) top_z = fmaxf(top_z, row[e]);
     top_z = warp_max(top_z);
@@ -138,7 +139,7 @@ __global__ void moe_route_grouped_kernel(const float* z, int tokens, int experts
             if (oe != 0x7fffffff && (best_e == 0x7fffffff || ov > best || (ov == best && oe < best_e))) { best = ov; best_e = oe; }
         }
         if ((best_e & 31) == lane) taken |= 1u << (best_e >> 5);
-        if (lane == 0) { ids[(size_t)warp * top + k] = best_e; weights[(size_t)warp * top + k] = score_of(best_e); }
+        if (lane == 0) { ids[(size_t)warp * top + k] = best_e; weights[(size_t)warp * top + k] = score_of(best_e) * scale; }
     }
 }
 
@@ -206,7 +207,7 @@ template <int MODE, bool GATHER>
 __global__ void __launch_bounds__(kGThreads)
 moe_grouped_mma_kernel(const bf16* A, int lda, const int* src_of, const float* weight_of, int top,
                        const bf16* W, long long w_stride, const int* tile_expert, const int* tile_row0,
-                       const int* n_tiles, const int* offsets, int N, int K, int act, int interleaved, void* C) {
+                       const int* n_tiles, const int* offsets, int N, int K, int act, GateConst gc, int interleaved, void* C) {
     __shared__ __align__(16) bf16 As[2][kGM][kGK + kGPad];
     __shared__ __align__(16) bf16 Bs[2][kGN][kGK + kGPad];
     constexpr bool GATED = MODE == 1;
@@ -321,8 +322,8 @@ moe_grouped_mma_kernel(const bf16* A, int lda, const int* src_of, const float* w
                     const int col = n0 + wn * 16 + ni * 8 + (lane & 3) * 2;
                     const float g0 = acc[mi][ni][hrow * 2], g1 = acc[mi][ni][hrow * 2 + 1];
                     const float u0 = acc[mi][ni + 2][hrow * 2], u1 = acc[mi][ni + 2][hrow * 2 + 1];
-                    if (col < N) out[col] = __float2bfloat16_rn(gate_act(g0, act) * u0);
-                    if (col + 1 < N) out[col + 1] = __float2bfloat16_rn(gate_act(g1, act) * u1);
+                    if (col < N) out[col] = __float2bfloat16_rn(gated_unit(g0, u0, act, gc));
+                    if (col + 1 < N) out[col + 1] = __float2bfloat16_rn(gated_unit(g1, u1, act, gc));
                 }
             } else if (MODE == 2) {
                 bf16* out = (bf16*)C + (size_t)(row0 + r) * N;
@@ -350,7 +351,7 @@ moe_grouped_mma_kernel(const bf16* A, int lda, const int* src_of, const float* w
 template <typename TA, int MODE, bool GATHER>
 __global__ void moe_grouped_plain_kernel(const TA* A, int lda, const int* src_of, const float* weight_of, int top,
                                          const TA* W, long long w_stride, const int* expert_of_row, int rows,
-                                         int N, int K, int act, int interleaved, int real, void* C) {
+                                         int N, int K, int act, GateConst gc, int interleaved, int real, void* C) {
     constexpr bool GATED = MODE == 1;
     TLLM_PDL_ENTER();
     const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -376,7 +377,7 @@ __global__ void moe_grouped_plain_kernel(const TA* A, int lda, const int* src_of
             g += x * to_f32<TA>(wg[k]);
             u += x * to_f32<TA>(wu[k]);
         }
-        ((TA*)C)[idx] = from_f32<TA>(gate_act(g, act) * u);
+        ((TA*)C)[idx] = from_f32<TA>(gated_unit(g, u, act, gc));
     } else {
         for (int k = 0; k < K; ++k) g += to_f32<TA>(from_f32<TA>(to_f32<TA>(a[k]) * w)) * to_f32<TA>(wg[k]);
         if (MODE == 2) ((TA*)C)[idx] = from_f32<TA>(gate_act(g, act));
@@ -404,17 +405,19 @@ __global__ void moe_gather_kernel(const bf16* x, const int* src_of, const float*
 
 // ---------------------------------------------------------------- combine
 // x, expert_of_row, real: where given, an assignment whose expert is `real` or later adds the token's own row
-// of x (times the weight) instead of a row of y.
+// of x (times the weight) instead of a row of y.  shared_gate: one logit per token, `ldsg` floats apart, whose sigmoid
+// multiplies the shared unit's output (null: it is added as it is).
 template <typename T, typename TY>
 __global__ void moe_combine_kernel(const TY* y, const int* row_of, const float* weight_of, int top,
                                    const T* shared, T* out, int width, size_t total, const T* x,
-                                   const int* expert_of_row, int real) {
+                                   const int* expert_of_row, int real, const float* shared_gate, int ldsg) {
     TLLM_PDL_ENTER();
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     const size_t stride = (size_t)gridDim.x * blockDim.x;
     for (; idx < total; idx += stride) {
         const size_t t = idx / width, i = idx - t * width;
         float v = shared != nullptr ? to_f32<T>(shared[idx]) : 0.0f;
+        if (shared_gate != nullptr) v *= 1.0f / (1.0f + expf(-shared_gate[t * ldsg]));
         for (int k = 0; k < top; ++k) {
             const int row = row_of[t * top + k];
             const float yv = (x != nullptr && expert_of_row[row] >= real) ? to_f32<T>(x[idx])
@@ -446,18 +449,19 @@ int tllm_moe_route(const float* z, int tokens, int experts, int top, int softmax
 
 // score_mode: 0 sigmoid(z), 1 softmax(z) over all experts.  correction [experts] float32 or null.  groups equal
 // groups of neighbouring experts, of which the `keep` with the best member may be chosen from.
-int tllm_moe_route_grouped(const float* z, int tokens, int experts, int top, int score_mode, const float* correction,
-                           int groups, int keep, int* ids, float* weights, cudaStream_t stream) {
+int tllm_moe_route_grouped(const float* z, int ldz, int tokens, int experts, int top, int score_mode, const float* correction,
+                           int groups, int keep, float scale, int* ids, float* weights, cudaStream_t stream) {
     TLLM_REQUIRE(tokens >= 0 && experts > 0 && experts <= 1024 && top > 0 && top <= experts,
                  "moe_route_grouped: %d experts, top %d", experts, top);
+    TLLM_REQUIRE(ldz >= experts, "moe_route_grouped: rows of %d for %d experts", ldz, experts);
     TLLM_REQUIRE(score_mode == 0 || score_mode == 1, "moe_route_grouped: unknown scores %d", score_mode);
     TLLM_REQUIRE(groups > 0 && experts % groups == 0 && keep > 0 && keep <= groups && keep * (experts / groups) >= top,
                  "moe_route_grouped: %d groups of %d experts, %d kept, top %d", groups, experts, keep, top);
     if (tokens == 0) return 0;
     const int warps = 4;
     launch_pdl(kPdlOther, moe_route_grouped_kernel, dim3((tokens + warps - 1) / warps), dim3(warps * 32),
-               (size_t)warps * (experts + groups) * sizeof(float), stream, z, tokens, experts, top, score_mode,
-               correction, groups, keep, ids, weights);
+               (size_t)warps * (experts + groups) * sizeof(float), stream, z, ldz, tokens, experts, top, score_mode,
+               correction, groups, keep, scale, ids, weights);
     return finish_launch("moe_route_grouped");
 }
 
@@ -477,9 +481,12 @@ int tllm_moe_plan(const int* ids, int n, int experts, int real, int tile_rows, i
 int tllm_moe_grouped(const void* A, int lda, const int* src_of, const float* weight_of, int top, const void* W,
                      long long w_stride, const int* tile_expert, const int* tile_row0, const int* n_tiles,
                      const int* offsets, const int* expert_of_row, int rows, int max_tiles, int N, int K,
-                     int dtype, int mode, int gather, int act, int interleaved, int real, void* C, cudaStream_t stream) {
+                     int dtype, int mode, int gather, int act, float limit, float slope, int interleaved, int real, void* C,
+                     cudaStream_t stream) {
+    const GateConst gc{limit, slope};
     const bool gated = mode == 1;
     TLLM_REQUIRE(mode >= 0 && mode <= 2, "moe_grouped: unknown mode %d", mode);
+    TLLM_REQUIRE(act != kActClampedSwish || (gated && limit > 0.0f), "moe_grouped: the clamped swish is a gated unit's with a positive limit");
     TLLM_REQUIRE(!interleaved || (gated && N % 8 == 0), "moe_grouped: interleaved gate and up rows need N %% 8 == 0");
     TLLM_REQUIRE(rows >= 0 && N > 0 && K > 0 && max_tiles > 0, "moe_grouped: bad sizes");
     TLLM_REQUIRE(dtype == kBF16 || dtype == kF32, "moe_grouped: unknown dtype %d", dtype);
@@ -491,7 +498,7 @@ int tllm_moe_grouped(const void* A, int lda, const int* src_of, const float* wei
         const dim3 grid((N + cols - 1) / cols, max_tiles), block(kGThreads);
 #define MMA(G, H)                                                                                              \
     launch_pdl(kPdlOther, moe_grouped_mma_kernel<G, H>, grid, block, 0, stream, (const bf16*)A, lda, src_of,    \
-               weight_of, top, (const bf16*)W, w_stride, tile_expert, tile_row0, n_tiles, offsets, N, K, act, interleaved, C)
+               weight_of, top, (const bf16*)W, w_stride, tile_expert, tile_row0, n_tiles, offsets, N, K, act, gc, interleaved, C)
         if (gated && gather) MMA(1, true);
         else if (gated) MMA(1, false);
         else if (mode == 2 && gather) MMA(2, true);
@@ -505,7 +512,7 @@ int tllm_moe_grouped(const void* A, int lda, const int* src_of, const float* wei
     const dim3 grid((unsigned)((total + 255) / 256)), block(256);
 #define PLAIN(T, G, H)                                                                                          \
     launch_pdl(kPdlOther, moe_grouped_plain_kernel<T, G, H>, grid, block, 0, stream, (const T*)A, lda, src_of,  \
-               weight_of, top, (const T*)W, w_stride, expert_of_row, rows, N, K, act, interleaved, real, C)
+               weight_of, top, (const T*)W, w_stride, expert_of_row, rows, N, K, act, gc, interleaved, real, C)
 #define PLAIN_T(T)                                         \
     do {                                                   \
         if (gated && gather) PLAIN(T, 1, true);            \
@@ -537,9 +544,10 @@ int tllm_moe_gather(const void* x, const int* src_of, const float* weight_of, in
 // x, expert_of_row, real: all or none; assignments to experts from `real` on add the token's row of x.
 int tllm_moe_combine(const void* y, int y_dtype, const int* row_of, const float* weight_of, int top, const void* shared,
                      void* out, int dtype, int tokens, int width, const void* x, const int* expert_of_row, int real,
-                     cudaStream_t stream) {
+                     const float* shared_gate, int ldsg, cudaStream_t stream) {
     TLLM_REQUIRE(tokens >= 0 && width > 0 && top > 0, "moe_combine: bad sizes");
     TLLM_REQUIRE(x == nullptr || expert_of_row != nullptr, "moe_combine: identity experts need the rows' experts");
+    TLLM_REQUIRE(shared_gate == nullptr || (shared != nullptr && ldsg > 0), "moe_combine: a gate without a shared unit");
     const size_t total = (size_t)tokens * width;
     if (total == 0) return 0;
     const int block = 256;
@@ -547,13 +555,13 @@ int tllm_moe_combine(const void* y, int y_dtype, const int* row_of, const float*
     const int grid = (int)(g > 148 * 16 ? 148 * 16 : g);
     if (dtype == kBF16 && y_dtype == kBF16)
         launch_pdl(kPdlOther, moe_combine_kernel<bf16, bf16>, dim3(grid), dim3(block), 0, stream, (const bf16*)y, row_of, weight_of, top,
-                   (const bf16*)shared, (bf16*)out, width, total, (const bf16*)x, expert_of_row, real);
+                   (const bf16*)shared, (bf16*)out, width, total, (const bf16*)x, expert_of_row, real, shared_gate, ldsg);
     else if (dtype == kBF16 && y_dtype == kF32)
         launch_pdl(kPdlOther, moe_combine_kernel<bf16, float>, dim3(grid), dim3(block), 0, stream, (const float*)y, row_of, weight_of, top,
-                   (const bf16*)shared, (bf16*)out, width, total, (const bf16*)x, expert_of_row, real);
+                   (const bf16*)shared, (bf16*)out, width, total, (const bf16*)x, expert_of_row, real, shared_gate, ldsg);
     else if (dtype == kF32 && y_dtype == kF32)
         launch_pdl(kPdlOther, moe_combine_kernel<float, float>, dim3(grid), dim3(block), 0, stream, (const float*)y, row_of, weight_of, top,
-                   (const float*)shared, (float*)out, width, total, (const float*)x, expert_of_row, real);
+                   (const float*)shared, (float*)out, width, total, (const float*)x, expert_of_row, real, shared_gate, ldsg);
     else
         TLLM_REQUIRE(false, "moe_combine: unknown dtypes %d, %d", dtype, y_dtype);
     return finish_launch("moe_combine");

@@ -66,11 +66,11 @@ def _declare(h) -> None:
         "tllm_qkv_unit_store": [vp, i32, vp, vp, f32, i32, vp, vp, vp, i32, i32, vp, vp, i64, vp, i32, i32,
                                 i32, i32, i32, i32, i32, vp, i32, f32, i32, i32, vp, vp],
         "tllm_attention_biased_general": [vp, vp, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32,
-                                          f32, f32, i32, i32, i32, vp, vp, vp, i32, i32, vp, i32, i32, vp, vp],
+                                          f32, f32, i32, i32, i32, vp, vp, vp, i32, i32, vp, i32, i32, i32, f32, f32, f32, vp, vp],
         "tllm_attention_biased_prefill": [vp, vp, vp, i64, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32,
-                                          f32, f32, i32, i32, i32, vp, vp, vp, i32, i32, vp, i32, i32, vp, vp],
+                                          f32, f32, i32, i32, i32, vp, vp, vp, i32, i32, vp, i32, i32, i32, f32, f32, f32, vp, vp],
         "tllm_attention_biased_decode": [vp, vp, vp, i64, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32,
-                                         f32, f32, i32, i32, i32, vp, vp, vp, i32, i32, vp, i32, i32, i32, vp, vp, vp],
+                                         f32, f32, i32, i32, i32, vp, vp, vp, i32, i32, vp, i32, i32, i32, f32, f32, f32, i32, vp, vp, vp],
         "tllm_scaled_add_layernorm": [vp, vp, vp, i32, vp, i32, f32, vp, i32, vp, i32, i32, vp],
         "tllm_linear_prepare": [vp, i32, i32, vp, i32, vp, i32, f32, vp, i32, i32, i32, f32, vp, vp, vp, vp, vp, vp,
                                 i32, vp],
@@ -80,7 +80,11 @@ def _declare(h) -> None:
         "tllm_activation": [vp, vp, i32, i32, i32, i32, vp, vp, i32, i32, i32, vp],
         "tllm_delta_prepare": [vp, i32, i32, vp, vp, i32, vp, i32, vp, vp, vp, vp, i64, i32, i32, i32, i32, f32, f32,
                                vp, vp, vp, vp, vp, i32, i32, i32, vp],
-        "tllm_delta_scan": [vp, i32, vp, vp, vp, vp, vp, vp, vp, i64, i32, i32, i32, i32, vp, i32, vp, i64, f32, vp, vp],
+        "tllm_delta_scan": [vp, i32, vp, vp, vp, vp, vp, vp, vp, i64, i32, i32, i32, i32, vp, i32, vp, vp, i64, f32, vp, vp],
+        "tllm_erase_prepare": [vp, i32, i32, i32, vp, i32, vp, vp, f32, vp, i32, i32, i32, f32, vp, vp, vp, vp, vp, i32, vp],
+        "tllm_stream_read": [vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, f32, vp, i32, vp, vp, vp, i64, i32, vp, vp, i32, i32, i32, vp],
+        "tllm_stream_tails": [vp, i32, vp, i32, vp, i64, i32, vp],
+        "tllm_embedding_sinusoid": [vp, vp, vp, i32, vp, f32, vp, i32, i32, i32, i32, vp],
         "tllm_delta_finish": [vp, vp, i32, i32, vp, f32, vp, i32, i32, i32, i32, i32, vp, i32, vp, i32, i32, vp, i64,
                               vp, i32, i32, vp],
         "tllm_latent_norm_store": [vp, i32, i32, i32, i32, i32, i32, vp, vp, f32, vp, f32, vp, vp, vp, i32, i32,
@@ -88,19 +92,19 @@ def _declare(h) -> None:
         "tllm_latent_query": [vp, i32, vp, i32, i32, i32, i32, i32, i32, vp, f32, vp, vp, i32, vp, i32, vp],
         "tllm_heads_gate": [vp, vp, i32, i32, i32, i32, i32, vp, vp, i32, vp],
         "tllm_moe_route": [vp, i32, i32, i32, i32, vp, vp, vp],
-        "tllm_moe_route_grouped": [vp, i32, i32, i32, i32, vp, i32, i32, vp, vp, vp],
+        "tllm_moe_route_grouped": [vp, i32, i32, i32, i32, i32, vp, i32, i32, f32, vp, vp, vp],
         "tllm_moe_plan": [vp, i32, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp],
         "tllm_moe_grouped": [vp, i32, vp, vp, i32, vp, i64, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32,
-                             i32, i32, i32, i32, vp, vp],
+                             i32, i32, f32, f32, i32, i32, vp, vp],
         "tllm_moe_gather": [vp, vp, vp, i32, vp, i32, i32, vp],
-        "tllm_moe_combine": [vp, i32, vp, vp, i32, vp, vp, i32, i32, i32, vp, vp, i32, vp],
+        "tllm_moe_combine": [vp, i32, vp, vp, i32, vp, vp, i32, i32, i32, vp, vp, i32, vp, i32, vp],
         "tllm_sum_rmsnorm": [vp, vp, vp, i32, f32, vp, vp, f32, vp, i32, i32, i32, vp],
         "tllm_ssd_prepare": [vp, i32, i32, vp, vp, vp, i32, vp, vp, vp, vp, i64, i64, i32, i32, i32, i32, vp, vp, vp,
                              vp, vp, i32, vp],
         "tllm_ssd_finish": [vp, vp, vp, i32, vp, i32, i32, vp, f32, i32, vp, i32, i32, i32, i32, vp, i64, i64, vp, vp],
-        "tllm_gemm_tcgen05_grouped": [vp, vp, vp, i32, i32, i32, i32, i32, vp, vp, vp, vp, i32, vp, vp],
+        "tllm_gemm_tcgen05_grouped": [vp, vp, vp, i32, i32, i32, i32, i32, vp, vp, vp, vp, i32, f32, f32, vp, vp],
         "tllm_add_rmsnorm": [vp, vp, vp, i32, f32, vp, i32, vp, i32, i32, vp],
-        "tllm_swiglu": [vp, vp, i32, i32, i32, i32, i32, vp],
+        "tllm_swiglu": [vp, vp, i32, i32, i32, i32, i32, f32, f32, vp],
         "tllm_cast": [vp, i32, vp, i32, i64, vp],
         "tllm_feed_tokens": [vp, vp, vp, vp, i32, vp],
         "tllm_qk_norm_rope_store": [vp, vp, vp, i32, f32, vp, i32, vp, vp, vp, i32, vp, i32, vp,
@@ -112,8 +116,8 @@ def _declare(h) -> None:
         "tllm_sample_split": [vp, i32, i32, i64, vp, vp, vp, vp, i32, vp, vp],
         "tllm_gemm_skinny": [vp, vp, vp, i32, i32, i32, i32, vp],
         "tllm_gemm_plain": [vp, i32, vp, i32, vp, i32, i32, i32, i32, vp],
-        "tllm_gemm_tcgen05": [vp, vp, vp, i32, i32, i32, i32, vp, vp],
-        "tllm_gemm_skinny_swiglu": [vp, vp, vp, i32, i32, i32, i32, vp],
+        "tllm_gemm_tcgen05": [vp, vp, vp, i32, i32, i32, i32, f32, f32, vp, vp],
+        "tllm_gemm_skinny_swiglu": [vp, vp, vp, i32, i32, i32, i32, f32, f32, vp],
         "tllm_gemm_skinny_act": [vp, vp, vp, i32, i32, i32, i32, vp],
         "tllm_paged_attention_decode": [vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32, f32,
                                         i32, vp, vp, vp, vp],
@@ -133,6 +137,8 @@ def _declare(h) -> None:
     h.tllm_delta_rule_state_floats.restype = i64
     h.tllm_attention_biased_fast_ok.argtypes = [i32, i32, i32, i32]
     h.tllm_attention_biased_fast_ok.restype = i32
+    h.tllm_attention_maps_fast_ok.argtypes = [i32, i32, i32, i32, i32]
+    h.tllm_attention_maps_fast_ok.restype = i32
     h.tllm_moe_tile_rows.argtypes = []
     h.tllm_moe_tile_rows.restype = i32
     h.tllm_paged_attention_prefill_tc_rows.argtypes = [i32, i32]
@@ -265,18 +271,28 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
     return torch.stack([gate.reshape(inter // 8, 8, k), up.reshape(inter // 8, 8, k)], dim=1).reshape(2 * inter, k)
 
 
-ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}      # codes of csrc/common.cuh (GateAct)
+ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 4}      # of gated units: codes of csrc/common.cuh (GateAct)
+NO_CONSTS = (0.0, 0.0)       # ``consts``: (limit, slope) of ``clamped_swish``, g sigmoid(slope g) (u + 1) with g = min(gate,
+                             # limit) and u = up held within -limit .. limit; the other activations have none
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, interleaved: bool = False, act: str = "silu") -> torch.Tensor:
+def _consts(act: str, consts):
+    limit, slope = NO_CONSTS if consts is None else consts
+    if act == "clamped_swish" and not limit > 0.0:
+        raise KernelError("clamped_swish needs its constants (limit, slope)")
+    return float(limit), float(slope)
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, interleaved: bool = False, act: str = "silu",
+           consts=None) -> torch.Tensor:
     """out[t, i] = act(gate) * up with gate = gate_up[t, i], up = gate_up[t, I + i], or, for columns
     interleaved by eight, gate = gate_up[t, 16 (i // 8) + i % 8] and up eight columns further.
-    ``act``: ``silu`` or ``gelu_tanh``."""
+    ``act``: ``silu``, ``gelu_tanh`` or ``clamped_swish`` (with its ``consts``)."""
     _cuda(gate_up, out)
     tokens, two_i = gate_up.shape
     assert out.shape == (tokens, two_i // 2) and out.dtype == gate_up.dtype
     _check(lib().tllm_swiglu(_p(gate_up), _p(out), _dt(out), tokens, two_i // 2, int(interleaved),
-                             ACTIVATIONS[act], _stream()), "swiglu")
+                             ACTIVATIONS[act], *_consts(act, consts), _stream()), "swiglu")
     return out
 
 
@@ -580,7 +596,7 @@ def tcgen05_pays(rows: int, out_cols: int, k: int, dtype, col_tile: int = 256) -
 
 
 def gemm_tcgen05(x: torch.Tensor, weight: torch.Tensor, swiglu: bool = False, short_tiles: bool = False,
-                 interleaved: bool = False, act: str = "silu", unary: bool = False) -> torch.Tensor:
+                 interleaved: bool = False, act: str = "silu", unary: bool = False, consts=None) -> torch.Tensor:
     """y = x . weight^T on tcgen05 tensor cores fed by TMA (csrc/gemm_tcgen05.cu), bfloat16 in
     and out, float32 accumulation in tensor memory.  With ``swiglu`` the weight is [gate; up]
     (or, ``interleaved``, gate and up rows interleaved by eight) and the result is
@@ -596,7 +612,8 @@ def gemm_tcgen05(x: torch.Tensor, weight: torch.Tensor, swiglu: bool = False, sh
     global tcgen05_calls
     tcgen05_calls += 1
     _check(lib().tllm_gemm_tcgen05(_p(x), _p(weight), _p(y), rows, n, k, int(swiglu) | (2 if short_tiles else 0) | (4 if interleaved else 0) | (16 if unary else 0)
-                                   | (ELEMENTWISE_ACTIVATIONS[act] << 8 if (swiglu or unary) else 0),
+                                   | ((ELEMENTWISE_ACTIVATIONS[act] if unary else ACTIVATIONS[act]) << 8 if (swiglu or unary) else 0),
+                                   *(_consts(act, consts) if swiglu else NO_CONSTS),
                                    _p(error_word(x.device)), _stream()), "gemm_tcgen05")
     return y
 
@@ -633,20 +650,20 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dtyp
     return torch.mm(x, weight.t(), out_dtype=want)
 
 
-def gemm_skinny_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, act: str = "silu") -> torch.Tensor:
+def gemm_skinny_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, act: str = "silu", consts=None) -> torch.Tensor:
     """silu(x . Wg^T) * (x . Wu^T) for at most 16 bfloat16 rows as one weight-streaming kernel;
     ``w_gate_up`` holds the rows of Wg and Wu interleaved by eight (``interleave_gate_up``)."""
     _cuda(x, w_gate_up)
     rows, k = x.shape
     inter = w_gate_up.shape[0] // 2
     out = torch.empty((rows, inter), dtype=torch.bfloat16, device=x.device)
-    _check(lib().tllm_gemm_skinny_swiglu(_p(x), _p(w_gate_up), _p(out), rows, inter, k, ACTIVATIONS[act], _stream()),
-           "gemm_skinny_swiglu")
+    _check(lib().tllm_gemm_skinny_swiglu(_p(x), _p(w_gate_up), _p(out), rows, inter, k, ACTIVATIONS[act],
+                                         *_consts(act, consts), _stream()), "gemm_skinny_swiglu")
     return out
 
 
 def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out_dtype: torch.dtype,
-                  interleaved: bool = False, act: str = "silu") -> torch.Tensor:
+                  interleaved: bool = False, act: str = "silu", consts=None) -> torch.Tensor:
     """silu(x . Wg^T) * (x . Wu^T) for w_gate_up = [Wg; Wu], or with the rows of Wg and Wu
     interleaved by eight (``interleave_gate_up``).  With enough bfloat16 rows the product and the
     activation are one tcgen05 kernel, with few rows and interleaved weights one weight-streaming
@@ -656,12 +673,12 @@ def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out_dtype: torch.dty
     plain = x.dtype == w_gate_up.dtype == out_dtype == torch.bfloat16 and x.is_contiguous() \
         and w_gate_up.is_contiguous()
     if plain and tcgen05_pays(rows, inter, k, w_gate_up.dtype, col_tile=128):
-        return gemm_tcgen05(x, w_gate_up, swiglu=True, interleaved=interleaved, act=act)
+        return gemm_tcgen05(x, w_gate_up, swiglu=True, interleaved=interleaved, act=act, consts=consts)
     if plain and interleaved and 0 < rows <= SKINNY_MAX_ROWS and k % 8 == 0:
-        return gemm_skinny_swiglu(x, w_gate_up, act)
+        return gemm_skinny_swiglu(x, w_gate_up, act, consts)
     gate_up = linear(x, w_gate_up, out_dtype=out_dtype)
     out = torch.empty((rows, inter), dtype=out_dtype, device=x.device)
-    return swiglu(gate_up, out, interleaved, act)
+    return swiglu(gate_up, out, interleaved, act, consts)
 
 
 # --------------------------------------------------------------------------- attention with a modified score
@@ -727,7 +744,7 @@ def attention_biased(q: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tens
                      sink: bool = False, slopes: Optional[torch.Tensor] = None,
                      gate: Optional[torch.Tensor] = None, ctx=None, sink_logits: Optional[torch.Tensor] = None,
                      values_in_keys: bool = False, distance_bias: Optional[torch.Tensor] = None,
-                     gate_per_head: bool = False) -> torch.Tensor:
+                     gate_per_head: bool = False, difference=None) -> torch.Tensor:
     """Attention of every row of ``q`` [T, q_heads * dk] over the keys of its own request, with the
     score s = (q . k) * scale changed in this order by whatever is given: ``softcap`` (s <- cap *
     tanh(s / cap)), ``slopes`` [q_heads] float32 (s <- s - slope * (pos - key pos)); keys j <= pos from
@@ -737,14 +754,19 @@ def attention_biased(q: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tens
     whose rows may be strided): out *= sigmoid(gate).  ``values_in_keys``: a value is the first ``dv`` elements of its key's row (``v_plane`` is
     not looked at), as in attention over compressed vectors that are key and, in part, value at once.
     ``distance_bias`` [q_heads, L] float32: entry [h, min(pos - key pos, L - 1)] is added to the score after
-    everything else (a learned bias by distance; it is not scaled)."""
+    everything else (a learned bias by distance; it is not scaled).
+    ``difference`` (lambda, eps, scale): two attention maps per head over the same values; ``q`` is [T, q_heads * 2 dk] and
+    a key 2 dk wide, head by head map 1 | map 2, and the result a1 - lambda a2, divided by its root mean square over dv
+    (``eps``) and times ``scale``."""
     _cuda(q, positions, token_slot, block_table, out, slopes, sink_logits, distance_bias)
     dist_len = 0
     if distance_bias is not None:
         assert distance_bias.dtype == torch.float32 and distance_bias.dim() == 2 and distance_bias.shape[0] == q_heads
         dist_len = distance_bias.shape[1]
     tokens = q.shape[0]
-    assert tuple(out.shape) == (tokens, q_heads * dv) and out.dtype == q.dtype
+    maps = 1 if difference is None else 2
+    assert tuple(out.shape) == (tokens, q_heads * dv) and out.dtype == q.dtype and q.shape[1] == q_heads * maps * dk
+    assert k_plane.shape[3] == maps * dk and (maps == 1 or not values_in_keys)
     kp, stride = _plane(k_plane)
     if values_in_keys:
         assert dv <= dk
@@ -763,23 +785,24 @@ def attention_biased(q: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tens
         assert slopes.dtype == torch.float32 and slopes.numel() == q_heads
     gate_ptr = None if gate is None else gate.data_ptr()
     mods = (float(scale), float(softcap or 0.0), int(chunk or 0), int(window or 0), int(bool(sink)), _p(slopes),
-            _p(sink_logits), _p(distance_bias), dist_len, v_row, gate_ptr, gate_stride, int(gate_per_head))
+            _p(sink_logits), _p(distance_bias), dist_len, v_row, gate_ptr, gate_stride, int(gate_per_head), maps,
+            *((0.0, 0.0, 0.0) if difference is None else (float(v) for v in difference)))
     consts = mods + (_p(out), _stream())
     # the plain score, or one changed only by a table of biases and a learned sink, at width 128 on both
     # sides: prompt portions go to the tcgen05 kernel of the plain cache, which reads the two planes
-    tcgen05 = PREFILL_TCGEN05 and dk == 128 and dv == 128 and not values_in_keys and not softcap and not chunk \
+    tcgen05 = PREFILL_TCGEN05 and dk == 128 and dv == 128 and maps == 1 and not values_in_keys and not softcap and not chunk \
         and slopes is None and gate is None and (sink_logits is not None or not sink) \
         and page_size % 16 == 0 and stride % 128 == 0 and q_heads <= 65535
     if BIASED_FAST and ctx is not None and ctx.pf_tiles is not None and ctx.tokens == tokens \
             and q.dtype == torch.bfloat16 and (gate_stride % 2 == 0 or gate_per_head) and v_row % 8 == 0 \
-            and lib().tllm_attention_biased_fast_ok(q_heads, kv_heads, dk, dv):
+            and lib().tllm_attention_maps_fast_ok(q_heads, kv_heads, dk, dv, maps):
         # one-token rows: keys read once per group of query heads; longer portions: tensor-core tiles
         if ctx.n_dec:
             reach = min(v for v in (chunk, window, ctx.max_context or 1 << 30) if v)
             splits = biased_decode_splits(ctx.n_dec, kv_heads, reach)
             part = None
             if splits > 1:
-                part = workspace(q.device, ctx.n_dec * q_heads * splits * (dv + 2))
+                part = workspace(q.device, ctx.n_dec * q_heads * maps * splits * (dv + 2))
             _check(lib().tllm_attention_biased_decode(
                 _p(q), kp, vp, stride, _p(positions), _p(token_slot), _p(ctx.dec_rows), ctx.n_dec, _p(block_table),
                 block_table.shape[1], page_size, q_heads, kv_heads, dk, dv, *mods, splits, _p(part), _p(out), _stream()),
@@ -808,14 +831,12 @@ def attention_biased(q: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tens
         return out
     _check(lib().tllm_attention_biased_general(
         _p(q), kp, vp, stride, _p(positions), _p(token_slot), _p(block_table), block_table.shape[1], page_size,
-        _dt(q), tokens, q_heads, kv_heads, dk, dv, float(scale), float(softcap or 0.0), int(chunk or 0),
-        int(window or 0), int(bool(sink)), _p(slopes), _p(sink_logits), _p(distance_bias), dist_len, v_row,
-        None if gate is None else gate.data_ptr(), gate_stride, int(gate_per_head), _p(out), _stream()), "attention_biased")
+        _dt(q), tokens, q_heads, kv_heads, dk, dv, *consts), "attention_biased")
     return out
 
 
 # --------------------------------------------------------------------------- stream, embedding with positions, activations
-ELEMENTWISE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "gelu_erf": 2, "relu2": 3}      # codes of csrc/common.cuh (GateAct); relu2 = max(x, 0)^2
+ELEMENTWISE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "gelu_erf": 2, "relu2": 3, "tanh": 5}      # codes of csrc/common.cuh (GateAct); relu2 = max(x, 0)^2
 
 
 def embedding_norm(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, scale: float = 1.0,
@@ -891,6 +912,65 @@ def activation(x: torch.Tensor, act: str, ids: Optional[torch.Tensor] = None, ta
     return out
 
 
+# --------------------------------------------------------------------------- several residual streams
+def embedding_sinusoid(ids: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, freq: torch.Tensor, scale: float,
+                       streams: int = 1) -> torch.Tensor:
+    """[T, streams * width] float32, every stream the same: table[ids[t]] * scale + the position's sinusoids (column 2 i
+    the sine, 2 i + 1 the cosine of position * frequency i).  ``freq`` [ceil(width / 2), 2] float32: a frequency and the
+    rest that rounding it left.  Rows with a negative id become zero."""
+    _cuda(ids, positions, table, freq)
+    vocab, width = table.shape
+    assert ids.dtype == positions.dtype == torch.int32 and freq.dtype == torch.float32 and tuple(freq.shape) == ((width + 1) // 2, 2)
+    out = torch.empty((ids.numel(), streams * width), dtype=torch.float32, device=ids.device)
+    _check(lib().tllm_embedding_sinusoid(_p(ids), _p(positions), _p(table), _dt(table), _p(freq), float(scale), _p(out),
+                                         ids.numel(), width, vocab, int(streams), _stream()), "embedding_sinusoid")
+    return out
+
+
+def stream_read(x: torch.Tensor, streams: int, gain: torch.Tensor, eps: float, dtype: torch.dtype,
+                w_in: Optional[torch.Tensor] = None, delta: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
+                w_out: Optional[torch.Tensor] = None, delta_bias: Optional[torch.Tensor] = None,
+                gate: Optional[torch.Tensor] = None, gate_bias: Optional[torch.Tensor] = None,
+                shift: Optional[torch.Tensor] = None, tail: Optional[torch.Tensor] = None, token_slot=None,
+                seg_info=None, single_tokens: bool = False, rows: Optional[torch.Tensor] = None):
+    """What stands between two sub-layers of a model with several residual streams ``x`` [T, streams * width] float32:
+
+    * the update that the last sub-layer left, if ``delta`` [T, width] (storage type) is given: with y = (delta +
+      delta_bias) * sigmoid(gate + gate_bias) (the biases float32 [width], ``gate`` logits in the storage type; each
+      only where given), x_t <- sum_s mix[s, t] x_s + w_out[t] y, all streams at once from the old ones;
+    * the next sub-layer's input h = gain * u / sqrt(mean(u^2) + eps), u = sum_t w_in[t] x_t (None: the plain sum);
+    * with ``shift`` [width] also h + (h' - h) * shift, h' the previous token's h (rounded to the storage type as it is),
+      which before a portion's first row comes from ``tail[slot]`` ([slots, width] float32), moved on to the portion's
+      last row.  ``single_tokens``: every portion is one token; otherwise ``seg_info`` [segments, 4] lists them.
+
+    Returns (x after the update (a new tensor; ``x`` itself without one), h, shifted h or None).  With ``rows`` (int32)
+    only h of those rows is made and the first entry is None."""
+    _cuda(x, gain, w_in, delta, mix, w_out, delta_bias, gate, gate_bias, shift, tail, token_slot, seg_info, rows)
+    tokens, width = x.shape[0], x.shape[1] // streams
+    assert x.dtype == gain.dtype == torch.float32 and x.shape[1] == streams * width and gain.numel() == width
+    for v, n in ((w_in, streams), (mix, streams * streams), (w_out, streams), (delta_bias, width), (gate_bias, width), (shift, width)):
+        assert v is None or (v.dtype == torch.float32 and v.numel() == n)
+    for v in (delta, gate):
+        assert v is None or (v.dtype == dtype and tuple(v.shape) == (tokens, width))
+    n = tokens if rows is None else rows.numel()
+    h = torch.empty((n, width), dtype=dtype, device=x.device)
+    if n == 0:                                  # nothing is wanted (an empty tensor has no address to tell apart from none)
+        return None, h, None
+    x_new = torch.empty_like(x) if delta is not None and rows is None else None
+    shifted = torch.empty_like(h) if shift is not None else None
+    assert shift is None or (tail is not None and tail.dtype == torch.float32 and tail.shape[1] == width and (single_tokens or seg_info is not None))
+    _check(lib().tllm_stream_read(
+        _p(x), _p(x_new), _p(delta), _p(delta_bias), _p(gate), _p(gate_bias), _p(mix), _p(w_out), _p(w_in), _p(gain), float(eps),
+        _p(h), _DT[dtype], _p(shift), _p(shifted), _p(tail), 0 if tail is None else tail.stride(0), int(single_tokens),
+        _p(token_slot), _p(rows), n, width, streams, _stream()), "stream_read")
+    if shift is not None and not single_tokens:
+        _check(lib().tllm_stream_tails(_p(seg_info), seg_info.shape[0], _p(h), _DT[dtype], _p(tail), tail.stride(0), width,
+                                       _stream()), "stream_tails")
+    if rows is not None:
+        return None, h, None
+    return (x if x_new is None else x_new), h, shifted
+
+
 # --------------------------------------------------------------------------- delta rule with channel-wise decay
 def delta_rule_state_floats(heads: int, kv_heads: int, dk: int, dv: int, taps: int) -> int:
     """Float32 words of one request's state: S of every head in the scan kernel's layout, then the
@@ -898,7 +978,7 @@ def delta_rule_state_floats(heads: int, kv_heads: int, dk: int, dv: int, taps: i
     return int(lib().tllm_delta_rule_state_floats(heads, kv_heads, dk, dv, taps))
 
 
-SCAN_DELTA, SCAN_PLAIN, SCAN_MEMORY, SCAN_HEAD_DECAY = 0, 1, 2, 3     # recurrences of the scan kernel (csrc/delta_rule.cu, ScanMode)
+SCAN_DELTA, SCAN_PLAIN, SCAN_MEMORY, SCAN_HEAD_DECAY, SCAN_ERASE = 0, 1, 2, 3, 4     # recurrences of the scan kernel (csrc/delta_rule.cu, ScanMode)
 GATE_ACTS = {"sigmoid": 0, "silu": 1}                # what the read-out is multiplied by: act(gate)
 
 
@@ -952,10 +1032,47 @@ def delta_rule(proj: torch.Tensor, conv_w: torch.Tensor, taps: int, a: torch.Ten
            "delta_prepare")
     segments = tokens if seg_info is None else seg_info.shape[0]
     _check(lib().tllm_delta_scan(_p(seg_info), segments, _p(token_slot), _p(qn), _p(kn), _p(vv), _p(decay), _p(beta),
-                                 _p(state), state.stride(0), heads, kv_heads, dk, dv, _p(o_raw), SCAN_DELTA, None, 0, 0.0,
+                                 _p(state), state.stride(0), heads, kv_heads, dk, dv, _p(o_raw), SCAN_DELTA, None, None, 0, 0.0,
                                  None, _stream()), "delta_scan")
     return _delta_finish(o_raw, gate, out_weight, False, eps, token_slot, tokens, heads, kv_heads, dk, dv, out_dtype,
                          proj, ld, taps, state, None, gate_act)
+
+
+def erase_delta_rule(proj: torch.Tensor, a_col: int, z: torch.Tensor, z_bias: torch.Tensor, a_bias: torch.Tensor,
+                     rate: float, gate: torch.Tensor, gate_act: str, out_weight: torch.Tensor, weight_per_head: bool,
+                     eps: float, token_slot: torch.Tensor, seg_info: Optional[torch.Tensor], state: torch.Tensor, heads: int,
+                     dk: int, dv: int, unit_eps: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """One step of the delta rule with a removal rate per head and key channel, for every row of ``proj`` [T, ...] =
+    r | k | v | ... in the storage type with the removal's logits at column ``a_col``: with u = k / sqrt(sum(k^2) +
+    ``unit_eps``) per head, w = exp(-``rate`` sigmoid(z + z_bias)) and a = sigmoid(logits + a_bias),
+    S <- diag(w) S - (a * u) (u^T S) + k v^T (both terms from the old S), o = S^T r, from ``state[slot]`` (float32,
+    updated in place).  ``z`` [T, heads * dk] float32, ``z_bias`` and ``a_bias`` [heads * dk] float32.  The read-out is
+    divided by its root mean square per head, times ``out_weight``, times ``gate_act``(``gate``), as in
+    ``linear_recurrence``.  Returns [T, heads * dv] in ``out_dtype``."""
+    _cuda(proj, z, z_bias, a_bias, out_weight, token_slot, seg_info, state)
+    tokens, ld = proj.shape
+    assert z.dtype == z_bias.dtype == a_bias.dtype == state.dtype == torch.float32 and state.dim() == 2
+    assert z.shape == (tokens, heads * dk) and z_bias.numel() == a_bias.numel() == heads * dk
+    assert state.shape[1] == delta_rule_state_floats(heads, heads, dk, dv, 1)
+    ws = workspace(proj.device, tokens * heads * (4 * dk + 2 * dv) + 32)
+    at = 0
+
+    def take(n):
+        nonlocal at
+        t = ws[at:at + tokens * n]
+        at += -(-tokens * n // 4) * 4
+        return t
+    qn, kn, decay, erase, vv, o_raw = (take(heads * dk), take(heads * dk), take(heads * dk), take(heads * dk),
+                                       take(heads * dv), take(heads * dv))
+    _check(lib().tllm_erase_prepare(_p(proj), ld, _dt(proj), int(a_col), _p(z), z.stride(0), _p(z_bias), _p(a_bias), float(rate),
+                                    _p(token_slot), heads, dk, dv, float(unit_eps), _p(qn), _p(kn), _p(vv), _p(decay),
+                                    _p(erase), tokens, _stream()), "erase_prepare")
+    segments = tokens if seg_info is None else seg_info.shape[0]
+    _check(lib().tllm_delta_scan(_p(seg_info), segments, _p(token_slot), _p(qn), _p(kn), _p(vv), _p(decay), None,
+                                 _p(state), state.stride(0), heads, heads, dk, dv, _p(o_raw), SCAN_ERASE, None, _p(erase), 0,
+                                 0.0, None, _stream()), "delta_scan")
+    return _delta_finish(o_raw, gate, out_weight, weight_per_head, eps, token_slot, tokens, heads, heads, dk, dv,
+                         out_dtype, None, 0, 1, state, None, gate_act)
 
 
 LINEAR_KINDS = {"channel_decay": 0, "log_gates": 1}      # csrc/delta_rule.cu, LinearKind
@@ -1012,7 +1129,7 @@ def linear_recurrence(proj: torch.Tensor, kind: str, z: torch.Tensor, z_bias: to
     aux_off = delta_rule_state_floats(heads, heads, dk, cols, 1) if memory else 0
     _check(lib().tllm_delta_scan(_p(seg_info), segments, _p(token_slot), _p(qn), _p(kn), _p(vv), _p(decay), _p(wgate),
                                  _p(state), state.stride(0), heads, heads, dk, cols, _p(o_raw),
-                                 SCAN_MEMORY if memory else SCAN_PLAIN, _p(fgate), aux_off, float(floor_eps), _p(den),
+                                 SCAN_MEMORY if memory else SCAN_PLAIN, _p(fgate), None, aux_off, float(floor_eps), _p(den),
                                  _stream()), "delta_scan")
     return _delta_finish(o_raw, gate, out_weight, weight_per_head, eps, token_slot, tokens, heads, heads, dk, dv,
                          out_dtype, None, 0, 1, state, den, gate_act)
@@ -1062,7 +1179,7 @@ def state_space(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: Optional[torch
     segments = tokens if seg_info is None else seg_info.shape[0]
     _check(lib().tllm_delta_scan(_p(seg_info), segments, _p(token_slot), _p(qn), _p(kn), _p(vv), None, _p(decay),
                                  _p(state), state.stride(0), heads, groups, n_state, head_dim, _p(o_raw), SCAN_HEAD_DECAY,
-                                 _p(step), 0, 0.0, None, _stream()), "delta_scan")
+                                 _p(step), None, 0, 0.0, None, _stream()), "delta_scan")
     out = torch.empty((tokens, inner), dtype=out_dtype, device=proj.device)
     _check(lib().tllm_ssd_finish(_p(o_raw), _p(vv), _p(skip), head_dim, _p(proj), ld, _dt(proj), _p(out_weight), float(eps),
                                  int(norm_groups), _p(token_slot), tokens, inner, channels, taps, _p(state),
@@ -1146,18 +1263,20 @@ ROUTER_SCORES = {"sigmoid": 0, "softmax": 1}      # scores over all experts (csr
 
 
 def moe_route_grouped(z: torch.Tensor, top: int, scores: str = "softmax", correction: Optional[torch.Tensor] = None,
-                      groups: int = 1, keep: int = 1):
+                      groups: int = 1, keep: int = 1, scale: float = 1.0, experts: Optional[int] = None):
     """(ids [T, top] int32, weights [T, top] float32) from float32 router logits ``z`` [T, E]: scores s over all E
     experts (``softmax`` or ``sigmoid``); the choice goes by s + ``correction`` ([E] float32, if given), within the
     ``keep`` of ``groups`` equal groups of neighbouring experts whose best member scores highest; the weights are
-    the chosen experts' s as they are.  Lowest index first on ties."""
+    the chosen experts' s, times ``scale``.  Lowest index first on ties.  ``experts``: how many of the row's columns are
+    logits (None: all; others may follow them)."""
     _cuda(z, correction)
-    assert z.dtype == torch.float32 and (correction is None or (correction.dtype == torch.float32 and correction.numel() == z.shape[1]))
-    tokens, experts = z.shape
+    tokens, ldz = z.shape
+    experts = ldz if experts is None else int(experts)
+    assert z.dtype == torch.float32 and (correction is None or (correction.dtype == torch.float32 and correction.numel() == experts))
     ids = torch.empty((tokens, top), dtype=torch.int32, device=z.device)
     weights = torch.empty((tokens, top), dtype=torch.float32, device=z.device)
-    _check(lib().tllm_moe_route_grouped(_p(z), tokens, experts, top, ROUTER_SCORES[scores], _p(correction), int(groups),
-                                        int(keep), _p(ids), _p(weights), _stream()), "moe_route_grouped")
+    _check(lib().tllm_moe_route_grouped(_p(z), ldz, tokens, experts, top, ROUTER_SCORES[scores], _p(correction), int(groups),
+                                        int(keep), float(scale), _p(ids), _p(weights), _stream()), "moe_route_grouped")
     return ids, weights
 
 
@@ -1201,18 +1320,19 @@ def moe_tcgen05_pays(rows: int, experts: int, n: int, k: int, dtype) -> bool:
 
 def moe_grouped(a: torch.Tensor, w: torch.Tensor, plan: MoePlan, top: int, gated: bool, gather: bool,
                 weights: Optional[torch.Tensor] = None, act: str = "silu", interleaved: bool = False,
-                out_dtype: Optional[torch.dtype] = None, unary: bool = False) -> torch.Tensor:
+                out_dtype: Optional[torch.dtype] = None, unary: bool = False, consts=None) -> torch.Tensor:
     """Per row r of the plan, A[r] . W[expert of r]^T.  ``w`` is [E, N (or 2 N: gate rows, then up rows, or
     ``interleaved`` by eight), K].  ``gather``: ``a`` is [tokens, K] and a row reads its token, times ``weights``
     [tokens, top] if given.  ``gated``: the result is act(gate) * up [rows, N] in the storage type, else
-    [rows, N] float32, or with ``unary`` act(.) [rows, N] in the storage type (``act`` then one of
+    [rows, N] float32 (``consts``: constants of ``act``, see ``ACTIVATIONS``), or with ``unary`` act(.) [rows, N] in the storage type (``act`` then one of
     ``ELEMENTWISE_ACTIVATIONS``).  A plan cut into tiles of 128 rows goes to the grouped tcgen05 product (bfloat16
     in and out; the gathered rows are laid out by a kernel of their own first).  Rows of experts without matrices
     (``plan.real``) are left unwritten."""
     _cuda(a, w, weights)
     experts, n_total, k = w.shape
     assert a.shape[1] == k and a.dtype == w.dtype and experts == plan.real and not (gated and unary)
-    act_code = ELEMENTWISE_ACTIVATIONS[act] if unary else ACTIVATIONS[act]
+    act_code = ELEMENTWISE_ACTIVATIONS[act] if unary else ACTIVATIONS[act] if gated else 0
+    limit, slope = _consts(act, consts) if gated else NO_CONSTS
     n = n_total // 2 if gated else n_total
     if plan.tile_rows == MOE_TCGEN05_TILE:
         assert a.dtype == torch.bfloat16 and (interleaved or not gated)
@@ -1227,31 +1347,36 @@ def moe_grouped(a: torch.Tensor, w: torch.Tensor, plan: MoePlan, top: int, gated
         flags = (1 | 4 | (act_code << 8)) if gated else ((16 | (act_code << 8)) if unary else 0)
         _check(lib().tllm_gemm_tcgen05_grouped(
             _p(a), _p(w), _p(out), plan.n, n_total, k, experts, flags, _p(plan.tile_expert), _p(plan.tile_row0),
-            _p(plan.n_tiles), _p(plan.offsets), plan.max_tiles, _p(error_word(a.device)), _stream()),
+            _p(plan.n_tiles), _p(plan.offsets), plan.max_tiles, limit, slope, _p(error_word(a.device)), _stream()),
             "gemm_tcgen05_grouped")
         return out
     out = torch.empty((plan.n, n), dtype=a.dtype if (gated or unary) else torch.float32, device=a.device)
     _check(lib().tllm_moe_grouped(
         _p(a), a.stride(0), _p(plan.src_of), _p(weights), top, _p(w), w.stride(0), _p(plan.tile_expert),
         _p(plan.tile_row0), _p(plan.n_tiles), _p(plan.offsets), _p(plan.expert_of_row), plan.n, plan.max_tiles,
-        n, k, _dt(a), 1 if gated else (2 if unary else 0), int(gather), act_code, int(interleaved), plan.real, _p(out),
+        n, k, _dt(a), 1 if gated else (2 if unary else 0), int(gather), act_code, limit, slope, int(interleaved), plan.real, _p(out),
         _stream()), "moe_grouped")
     return out
 
 
 def moe_combine(y: torch.Tensor, plan: MoePlan, top: int, shared: Optional[torch.Tensor], dtype: torch.dtype,
-                weights: Optional[torch.Tensor] = None, identity_input: Optional[torch.Tensor] = None) -> torch.Tensor:
+                weights: Optional[torch.Tensor] = None, identity_input: Optional[torch.Tensor] = None,
+                shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[t] = shared[t] + sum_k (weights[t, k] *) y[row of (t, k)], float32 sums, stored as ``dtype``;
     ``y`` float32 or in the storage type.  ``identity_input`` [T, width] (``dtype``): an assignment to an expert
-    without matrices (``plan.real`` or later) adds the token's row of it instead of a row of ``y``."""
+    without matrices (``plan.real`` or later) adds the token's row of it instead of a row of ``y``.
+    ``shared_gate`` [T] float32 (may be strided): the shared unit's output is multiplied by its sigmoid."""
     _cuda(y, shared, weights, identity_input)
     if identity_input is not None:
         assert identity_input.dtype == dtype and tuple(identity_input.shape) == (plan.n // top, y.shape[1])
     tokens, width = plan.n // top, y.shape[1]
     out = torch.empty((tokens, width), dtype=dtype, device=y.device)
+    if shared_gate is not None:
+        assert shared is not None and shared_gate.dtype == torch.float32 and tuple(shared_gate.shape) == (tokens,)
     if shared is not None:
         assert shared.dtype == dtype and tuple(shared.shape) == (tokens, width)
     _check(lib().tllm_moe_combine(_p(y), _dt(y), _p(plan.row_of), _p(weights), top, _p(shared), _p(out), _DT[dtype],
-                                  tokens, width, _p(identity_input), _p(plan.expert_of_row), plan.real, _stream()),
-           "moe_combine")
+                                  tokens, width, _p(identity_input), _p(plan.expert_of_row), plan.real,
+                                  None if shared_gate is None else shared_gate.data_ptr(),
+                                  0 if shared_gate is None else shared_gate.stride(0), _stream()), "moe_combine")
     return out

@@ -18,6 +18,10 @@ softmax, with an output gate.  Every step is a parameter, so other designs can p
               ``learned_sink`` exp(z_h) instead, z_h a learned number per head (tensor ``sink``)
   gate        ``output_gate``: the concatenated heads are multiplied by sigmoid(Wg x), x the mixer's input; with
               ``gate_per_head`` Wg has one row per head and a head is multiplied by one number
+  difference  ``differential`` (diff, eps): two attention maps per head over the same values.  q has q_heads * 2 and k
+              kv_heads * 2 vectors of width key_dim, head by head map 1 | map 2; with the maps' outputs a1, a2 and
+              lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff (four learned vectors of width key_dim, tensors
+              ``difference_names``) the head is o = a1 - lambda a2, then o / sqrt(mean(o^2) + eps) (1 - diff)
   biases      ``biases``: q, k, v and the output product have biases (tensors ``<name>`` + ``bias_suffix``), added in
               float32 where the norm kernel reads the projections; the output's is added by the product, or, with
               ``defer_output_bias``, left as ``deferred_bias`` for the block's sum kernel to add
@@ -64,6 +68,7 @@ def distance_buckets(rows: int, far: float) -> List[int]:
 class BiasedAttention:
     graph_safe = True
     NAMES = ("q", "k", "v", "o", "g")
+    DIFFERENCE_NAMES = ("lq1", "lk1", "lq2", "lk2")
 
     def __init__(self, hidden_size: int, q_heads: int, kv_heads: int, key_dim: int, value_dim: int,
                  scale: float, dtype: torch.dtype, device, unit_norm_eps: Optional[float] = None,
@@ -75,7 +80,8 @@ class BiasedAttention:
                  q_temperature: Optional[Tuple[float, int]] = None,
                  distance_bias: Optional[Tuple[int, float]] = None, bias_name: str = "rel",
                  learned_sink: bool = False, sink_name: str = "sink", gate_per_head: bool = False,
-                 biases: bool = False, bias_suffix: str = ".b", defer_output_bias: bool = False):
+                 biases: bool = False, bias_suffix: str = ".b", defer_output_bias: bool = False,
+                 differential: Optional[Tuple[float, float]] = None, difference_names: Sequence[str] = DIFFERENCE_NAMES):
         if q_heads % kv_heads:
             raise ValueError(f"{q_heads} query heads cannot share {kv_heads} key/value heads")
         if unit_norm_eps is not None and not unit_norm_eps > 0.0:
@@ -130,6 +136,14 @@ class BiasedAttention:
         self.defer_output_bias = bool(defer_output_bias) and self.biases
         if self.gate_per_head and not self.output_gate:
             raise ValueError("a gate per head is an output gate: give output_gate=True")
+        self.maps, self.differential, self.difference_names = 1, None, tuple(difference_names)
+        if differential is not None:
+            self.maps, self.differential = 2, (float(differential[0]), float(differential[1]))
+            if unit_norm_eps is not None or position is not None or self.values_are_keys:
+                raise ValueError("two maps per head come without head norms, rotation and keys as values")
+            if not self.differential[1] > 0.0:
+                raise ValueError("the difference of two maps is normed: its eps must be positive")
+        self.difference = None
         self.in_bias = self.out_bias = self.deferred_bias = None
         self.q_gain = self.k_gain = self.bias_table = self.sink_logits = None
         self.w_in = self.w_o = None
@@ -139,11 +153,12 @@ class BiasedAttention:
     def param_specs(cls, hidden_size, q_heads, kv_heads, key_dim, value_dim, output_gate=False,
                     names=NAMES, qk_gains=False, gain_suffix=".norm", values_are_keys=False, distance_bias=None,
                     bias_name="rel", learned_sink=False, sink_name="sink", gate_per_head=False, biases=False,
-                    bias_suffix=".b", **_) -> Dict[str, ParamSpec]:
+                    bias_suffix=".b", differential=None, difference_names=DIFFERENCE_NAMES, **_) -> Dict[str, ParamSpec]:
         q, k, v, o, g = names
+        maps = 1 if differential is None else 2
         specs = {
-            q: ParamSpec((q_heads * key_dim, hidden_size)),
-            k: ParamSpec((kv_heads * key_dim, hidden_size)),
+            q: ParamSpec((q_heads * maps * key_dim, hidden_size)),
+            k: ParamSpec((kv_heads * maps * key_dim, hidden_size)),
             o: ParamSpec((hidden_size, q_heads * value_dim)),
         }
         if not values_are_keys:
@@ -160,6 +175,8 @@ class BiasedAttention:
             specs[bias_name] = ParamSpec((int(distance_bias[0]), q_heads), "unit")
         if learned_sink:
             specs[sink_name] = ParamSpec((q_heads,), "unit")
+        if differential is not None:
+            specs.update({n: ParamSpec((key_dim,), "small") for n in difference_names})
         return specs
 
     def load(self, t: Dict[str, torch.Tensor]) -> None:
@@ -188,6 +205,11 @@ class BiasedAttention:
             self.bias_table = rel[index].t().contiguous()
         if self.learned_sink:
             self.sink_logits = t[self.sink_name].to(torch.float32).contiguous()
+        if self.differential is not None:
+            diff, eps = self.differential
+            a, b, c, d = (t[n].to(torch.float32) for n in self.difference_names)
+            lam = torch.exp((a * b).sum()) - torch.exp((c * d).sum()) + diff
+            self.difference = (float(lam), eps, 1.0 - diff)
 
     # ---- what the cache manager has to provide
     def reach(self) -> Optional[int]:
@@ -196,34 +218,35 @@ class BiasedAttention:
         return min(limits) if limits else None
 
     def cache_spec(self) -> Optional[CacheSpec]:
-        return CacheSpec(((self.kv_heads, self.dk), (self.kv_heads, self.dv)), self.reach())
+        return CacheSpec(((self.kv_heads, self.maps * self.dk), (self.kv_heads, self.dv)), self.reach())
 
     def state_spec(self) -> Optional[StateSpec]:
         return None
 
     def workspace_floats(self, tokens: int) -> int:
-        width_in = (self.q_heads + self.kv_heads) * self.dk + (self.kv_heads + 2 * self.q_heads) * self.dv
-        return tokens * (width_in + self.q_heads * self.dk)
+        width_in = (self.q_heads + self.kv_heads) * self.maps * self.dk + (self.kv_heads + 2 * self.q_heads) * self.dv
+        return tokens * (width_in + self.q_heads * self.maps * self.dk)
 
     # ---- one step
     def forward(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
         tokens = x.shape[0]
         proj = ops.linear(x, self.w_in, out_dtype=self.dtype)
-        q = torch.empty((tokens, self.q_heads * self.dk), dtype=self.dtype, device=x.device)
+        dk = self.maps * self.dk                      # a query head and a cached key hold every map's vector
+        q = torch.empty((tokens, self.q_heads * dk), dtype=self.dtype, device=x.device)
         k_plane, v_plane = cache.planes
         ops.qkv_unit_store(proj, q, ctx.positions, ctx.token_slot, cache.block_table, k_plane, v_plane,
-                           cache.page_size, self.q_heads, self.kv_heads, self.dk, self.dv,
+                           cache.page_size, self.q_heads, self.kv_heads, dk, self.dv,
                            self.unit_norm_eps, q_gain=self.q_gain, k_gain=self.k_gain, store=cache.writes,
                            inv_freq=self.inv_freq, rot_dims=self.rot_dims, q_temperature=self.q_temperature,
                            values_are_keys=self.values_are_keys, bias=self.in_bias)
         gate = None
         if self.output_gate:
-            at = (self.q_heads + self.kv_heads) * self.dk + (0 if self.values_are_keys else self.kv_heads * self.dv)
+            at = (self.q_heads + self.kv_heads) * dk + (0 if self.values_are_keys else self.kv_heads * self.dv)
             gate = proj[:, at:at + (self.q_heads if self.gate_per_head else self.q_heads * self.dv)]
         out = torch.empty((tokens, self.q_heads * self.dv), dtype=self.dtype, device=x.device)
         ops.attention_biased(q, k_plane, v_plane, ctx.positions, ctx.token_slot, cache.block_table,
                              cache.page_size, self.q_heads, self.kv_heads, self.dk, self.dv, self.scale, out,
                              softcap=self.softcap or 0.0, chunk=self.chunk or 0, window=self.window or 0,
                              sink=self.sink, slopes=self.slopes, gate=gate, ctx=ctx, sink_logits=self.sink_logits,
-                             distance_bias=self.bias_table, gate_per_head=self.gate_per_head)
+                             distance_bias=self.bias_table, gate_per_head=self.gate_per_head, difference=self.difference)
         return ops.linear(out, self.w_o, out_dtype=self.dtype, bias=self.out_bias)

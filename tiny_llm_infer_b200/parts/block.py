@@ -31,6 +31,12 @@ mixer (``postnorm_mixer``, ``postnorm_mixer_ffn``) or two side by side with weig
 ``postnorm_pair_ffn``, roles ``left`` and ``right``).  Every sum with its norm is one kernel (``RMSNorm.of_sum``),
 which also leaves the stream in the storage type; it travels from block to block as a ``StreamCopy``.  A mixer
 that says ``deferred_bias`` (a bias of its output product that it has not added) gets it added in that kernel.
+
+``hyper_*``: several residual streams (``parts/streams.py``).  Per sub-layer, u = sum_s in[s] x_s, y = sub-layer(norm(u)),
+x_t <- sum_s mix[s, t] x_s + out[t] y, for the mixer and, where the layer has one, the feed-forward: ``hyper_mixer``,
+``hyper_mixer_ffn``.  With ``_gated`` every output is multiplied by a residual gate of the norm's output, with
+``_shifted`` the mixer's input is shifted by a token (``hyper_mixer_ffn_gated_shifted`` and so on).  The last update goes on
+as a ``StreamUpdate``, which the next layer's first norm, or the model's last, applies.
 """
 from __future__ import annotations
 
@@ -41,6 +47,7 @@ import torch
 from .. import ops
 from .norm import NormedDelta, ScaledDeltas, StreamCopy
 from .registry import register
+from .streams import StreamUpdate
 
 
 class Block:
@@ -223,3 +230,49 @@ def _postnorm_block(name: str, mixer_roles, with_ffn: bool) -> type:
 for _roles, _name in ((("mixer",), "postnorm_mixer"), (("left", "right"), "postnorm_pair")):
     for _ffn in (False, True):
         _postnorm_block(_name + ("_ffn" if _ffn else ""), _roles, _ffn)
+
+
+def _hyper_block(name: str, with_ffn: bool, gated: bool, shifted: bool) -> type:
+    roles = {"norm1": "norm", "hc1": "norm"}
+    if shifted:
+        roles["shift"] = "mixer"
+    if gated:
+        roles["gate1"] = "norm"
+    roles["mixer"] = "mixer"
+    if with_ffn:
+        roles.update({"norm2": "norm", "hc2": "norm", "ffn": "feed_forward"})
+        if gated:
+            roles["gate2"] = "norm"
+
+    class HyperBlock(Block):
+        def _leave(self, x: torch.Tensor, h: torch.Tensor, y: torch.Tensor, part, mix, gate) -> StreamUpdate:
+            """The output ``y`` of ``part``, which read the norm's output ``h``, still to be mixed into the streams ``x``."""
+            update = StreamUpdate(x, y, getattr(part, "deferred_bias", None), mix=mix)
+            if gate is not None:
+                update.gate, update.gate_bias = gate.forward(h), gate.bias
+            return update
+
+        def forward(self, h: torch.Tensor, pending, ctx, cache) -> StreamUpdate:
+            if pending is not None and not isinstance(pending, StreamUpdate):
+                raise TypeError(f"a block over several streams cannot follow one that hands on a {type(pending).__name__}")
+            update = StreamUpdate(h) if pending is None else pending
+            views = cache if isinstance(cache, (list, tuple)) else [cache]
+            x, n, s = self.norm1.read(update, self.hc1, ctx, self.shift if shifted else None,
+                                      views[0].state if shifted else None)
+            update = self._leave(x, n, self.mixer.forward(s, ctx, views[-1]), self.mixer, self.hc1,
+                                 self.gate1 if gated else None)
+            if with_ffn:
+                x, n, _ = self.norm2.read(update, self.hc2)
+                update = self._leave(x, n, self.ffn.forward(n, ctx), self.ffn, self.hc2, self.gate2 if gated else None)
+            return update
+
+    HyperBlock.roles = roles
+    HyperBlock.__name__ = HyperBlock.__qualname__ = "".join(w.title() for w in name.split("_")) + "Block"
+    return register("block", name)(HyperBlock)
+
+
+for _ffn in (False, True):
+    for _gated in (False, True):
+        for _shifted in (False, True):
+            _hyper_block("hyper_mixer" + ("_ffn" if _ffn else "") + ("_gated" if _gated else "")
+                         + ("_shifted" if _shifted else ""), _ffn, _gated, _shifted)

@@ -22,9 +22,20 @@ dt_bias)) with Wa [heads, hidden] and no low rank (the kernels spread it over th
 
 Products: one for q | k | v | beta, one for the two low ranks (a1 | g1), one for both second halves (a
 block-diagonal weight, float32 result), one for the output; three kernels in between (``ops.delta_rule``).
+
+``erase_delta`` is the rule with a removal rate per head and key channel instead of one write strength, and no
+convolution: r, k = x Wr^T, x Wk^T (heads x dk), v = x Wv^T (heads x dv), u = k / sqrt(sum(k^2) + ``unit_eps``) per head,
+
+  w       = exp(-``decay_rate`` sigmoid(tanh(x W1^T) W2^T + w0)),   a = sigmoid(x Wa^T + ba), one each per head and channel
+  S      <- diag(w) S - (a * u) (u^T S) + k v^T, both terms from the old S;   o = S^T r
+  out     = (o / rms(o) per head * w_norm (heads x dv) * sigmoid(x Wg^T)) Wo^T
+
+Products: one for r | k | v | gate | a, one for the low rank with tanh in its epilogue, one for its second half
+(float32 result), one for the output.
 """
 from __future__ import annotations
 
+import math
 from typing import Dict, Optional, Sequence
 
 import torch
@@ -166,4 +177,64 @@ class ChannelDeltaRule:
                              self.out_weight, self.norm_eps, ctx.token_slot, ctx.seg_info, cache.state, self.heads,
                              self.kv_heads, self.dk, self.dv, self.dk ** -0.5, self.unit_eps, self.dtype, conv_t=self.conv_t,
                              decay_per_head=self.decay_per_head, beta_col=self.beta_col, gate_act=self.gate_act)
+        return ops.linear(out, self.w_o, out_dtype=self.dtype)
+
+
+@register("mixer", "erase_delta")
+class EraseDeltaRule:
+    graph_safe = True
+    NAMES = ("r", "k", "v", "g", "a", "w1", "w2", "w0", "norm", "o")
+
+    def __init__(self, hidden_size: int, heads: int, key_dim: int, value_dim: int, decay_rank: int, norm_eps: float,
+                 dtype: torch.dtype, device, decay_rate: float = math.exp(-0.5), unit_eps: float = 1e-6,
+                 gate_act: str = "sigmoid", bias_suffix: str = ".b", names: Sequence[str] = NAMES):
+        if -(-key_dim // scan_lanes(key_dim)) > SCAN_MAX_ROWS:
+            raise ValueError(f"keys of width {key_dim} are wider than the scan kernel takes ({32 * SCAN_MAX_ROWS})")
+        self.hidden, self.heads, self.dk, self.dv, self.decay_rank = hidden_size, heads, key_dim, value_dim, int(decay_rank)
+        self.norm_eps, self.unit_eps, self.decay_rate = float(norm_eps), float(unit_eps), float(decay_rate)
+        self.dtype, self.device, self.gate_act = dtype, device, gate_act
+        self.bias_suffix, self.names = bias_suffix, tuple(names)
+
+    # ---- weights
+    @classmethod
+    def param_specs(cls, hidden_size, heads, key_dim, value_dim, decay_rank, bias_suffix: str = ".b", names=NAMES,
+                    **_) -> Dict[str, ParamSpec]:
+        r, k, v, g, a, w1, w2, w0, norm, o = names
+        qk, vd = heads * key_dim, heads * value_dim
+        return {r: ParamSpec((qk, hidden_size)), k: ParamSpec((qk, hidden_size)), v: ParamSpec((vd, hidden_size)),
+                g: ParamSpec((vd, hidden_size)), a: ParamSpec((qk, hidden_size)), a + bias_suffix: ParamSpec((qk,), "unit"),
+                w1: ParamSpec((decay_rank, hidden_size)), w2: ParamSpec((qk, decay_rank)), w0: ParamSpec((qk,), "unit"),
+                norm: ParamSpec((vd,), "norm"), o: ParamSpec((hidden_size, vd))}
+
+    def load(self, t: Dict[str, torch.Tensor]) -> None:
+        r, k, v, g, a, w1, w2, w0, norm, o = self.names
+        parts = [t[r], t[k], t[v], t[g], t[a]]
+        pad = torch.zeros((-sum(p.shape[0] for p in parts) % 8, self.hidden), dtype=t[r].dtype, device=t[r].device)
+        self.w_in = torch.cat(parts + [pad], dim=0).contiguous()
+        self.gate_col = self.heads * (2 * self.dk + self.dv)
+        self.a_col = self.gate_col + self.heads * self.dv
+        self.w_1, self.w_2 = t[w1].contiguous(), t[w2].contiguous()
+        self.z_bias = t[w0].to(torch.float32).contiguous()
+        self.a_bias = t[a + self.bias_suffix].to(torch.float32).contiguous()
+        self.out_weight = t[norm].to(torch.float32).contiguous()
+        self.w_o = t[o].contiguous()
+
+    # ---- what the cache manager has to provide
+    def cache_spec(self) -> Optional[CacheSpec]:
+        return None
+
+    def state_spec(self) -> Optional[StateSpec]:
+        return StateSpec((state_floats(self.heads, self.heads, self.dk, self.dv, 1),), "float32")
+
+    def workspace_floats(self, tokens: int) -> int:
+        return tokens * self.heads * (8 * self.dk + 5 * self.dv)
+
+    # ---- one step
+    def forward(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
+        proj = ops.linear(x, self.w_in, out_dtype=self.dtype)
+        z = ops.linear(ops.linear_act(x, self.w_1, "tanh", self.dtype), self.w_2, out_dtype=torch.float32)
+        gate = proj[:, self.gate_col:self.a_col]
+        out = ops.erase_delta_rule(proj, self.a_col, z, self.z_bias, self.a_bias, self.decay_rate, gate, self.gate_act,
+                                   self.out_weight, True, self.norm_eps, ctx.token_slot, ctx.seg_info, cache.state,
+                                   self.heads, self.dk, self.dv, self.unit_eps, self.dtype)
         return ops.linear(out, self.w_o, out_dtype=self.dtype)

@@ -91,6 +91,37 @@ class TokenPositionEmbedding:
                                   self.norm_eps or 0.0)
 
 
+@register("embedding", "sinusoid_embedding")
+class SinusoidEmbedding:
+    """h0[t] = E[token[t]] * scale + S(position[t]), S(p)[2 i] = sin(p base^(-2 i / width)), S(p)[2 i + 1] the cosine of the
+    same; with ``streams`` > 1 the row starts as that many copies side by side, [T, streams * width].  No table bounds the
+    positions."""
+    takes_context = True
+
+    def __init__(self, vocab_size: int, hidden_size: int, dtype: torch.dtype, device, scale: float = 1.0, name: str = "weight",
+                 base: float = 10000.0, streams: int = 1):
+        self.vocab, self.hidden, self.dtype, self.device = vocab_size, hidden_size, dtype, device
+        self.scale, self.name, self.streams = float(scale), name, int(streams)
+        exact = float(base) ** (-2.0 * torch.arange((hidden_size + 1) // 2, dtype=torch.float64) / hidden_size)
+        rounded = exact.to(torch.float32)
+        rest = (exact - rounded.to(torch.float64)).to(torch.float32)
+        self.freq = torch.stack([rounded, rest], dim=1).contiguous().to(device)
+        self.weight: Optional[torch.Tensor] = None
+
+    @classmethod
+    def param_specs(cls, vocab_size, hidden_size, scale: float = 1.0, name: str = "weight", base: float = 10000.0,
+                    streams: int = 1) -> Dict[str, ParamSpec]:
+        return {name: ParamSpec((vocab_size, hidden_size))}
+
+    def load(self, t: Dict[str, torch.Tensor]) -> None:
+        self.weight = t[self.name].contiguous()
+
+    def forward(self, token_ids: torch.Tensor, ctx=None) -> torch.Tensor:
+        if ctx is None:
+            raise ValueError("an embedding with positions needs the step's context")
+        return ops.embedding_sinusoid(token_ids, ctx.positions, self.weight, self.freq, self.scale, self.streams)
+
+
 @register("head", "lm_head")
 class LMHead:
     def __init__(self, vocab_size: int, hidden_size: int, tied: bool, dtype: torch.dtype, device,

@@ -1,6 +1,8 @@
 """Dense gated feed-forward: d = (act(x Wg^T) * (x Wu^T)) Wd^T, no biases, act in float32:
 silu(g) = g / (1 + exp(-g)) (SwiGLU; reference: model/src/qwen3_paged_batch.cpp:281-295,
-kernels/src/swiglu_kernel_cpu.cpp:20-24) or, by the ``activation`` parameter, the tanh form of GELU.
+kernels/src/swiglu_kernel_cpu.cpp:20-24) or, by the ``activation`` parameter, the tanh form of GELU or the clamped
+swish, g sigmoid(slope g) (u + 1) with g = min(gate, limit) and u = up held within -limit .. limit (``act_consts`` =
+(limit, slope)).
 ``names`` are the checkpoint's names of the gate, up and down matrices behind the part's prefix.  Gate and up projections are one product with
 one weight of 2 I rows, fused at load time: eight rows of Wg, the eight rows of Wu that belong
 to them, and so on (``ops.interleave_gate_up``), so that a gate and its up meet in one
@@ -22,15 +24,16 @@ class SwiGLUFeedForward:
     NAMES = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
 
     def __init__(self, hidden_size: int, intermediate_size: int, dtype: torch.dtype, device,
-                 activation: str = "silu", names=NAMES):
+                 activation: str = "silu", names=NAMES, act_consts=None):
         if activation not in ops.ACTIVATIONS:
             raise ValueError(f"activation {activation!r} is not one of {sorted(ops.ACTIVATIONS)}")
         self.hidden, self.inter, self.dtype, self.device = hidden_size, intermediate_size, dtype, device
-        self.activation, self.names = activation, tuple(names)
+        self.activation, self.names, self.act_consts = activation, tuple(names), act_consts
         self.w_gate_up = self.w_down = None
 
     @classmethod
-    def param_specs(cls, hidden_size, intermediate_size, activation: str = "silu", names=NAMES) -> Dict[str, ParamSpec]:
+    def param_specs(cls, hidden_size, intermediate_size, activation: str = "silu", names=NAMES,
+                    act_consts=None) -> Dict[str, ParamSpec]:
         gate, up, down = names
         return {
             gate: ParamSpec((intermediate_size, hidden_size)),
@@ -53,7 +56,7 @@ class SwiGLUFeedForward:
 
     def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
         act = ops.linear_swiglu(x, self.w_gate_up, out_dtype=self.dtype, interleaved=self.interleaved,
-                                act=self.activation)
+                                act=self.activation, consts=self.act_consts)
         return ops.linear(act, self.w_down, out_dtype=self.dtype)
 
 

@@ -16,6 +16,10 @@ Options that other routers use, each a parameter:
                          best member's choice score is largest can be chosen
   ``identity``           the router's last ``identity`` outputs are experts without matrices whose output is their
                          input; they count as experts for the scores, the groups and the choice
+  ``router_scale``       the weights are multiplied by this number
+  ``act_consts``         constants of the experts' activation (``clamped_swish``: limit, slope)
+  ``shared_gate``        name of one more row [1, hidden] behind the shared unit's prefix: the unit's output is multiplied
+                         by the sigmoid of that product, one number per token (the row rides along in the router's product)
 
 The step's rows are sorted by expert on the device (``ops.MoePlan``); the experts' gate|up product
 gathers its rows from the tokens and applies the activation in its epilogue, the down product leaves
@@ -43,7 +47,8 @@ class MixtureOfExperts:
                  activation: str = "silu", router_scores: str = "sigmoid", weight_on: str = "input",
                  shared: Optional[PartSpec] = None, router_name: str = "router", expert_prefix: str = "e",
                  names=("gate", "up", "down"), gated: bool = True, correction: bool = False,
-                 correction_name: str = "correction", groups=None, identity: int = 0):
+                 correction_name: str = "correction", groups=None, identity: int = 0, router_scale: float = 1.0,
+                 act_consts=None, shared_gate: Optional[str] = None):
         if not 0 < top <= experts + identity:
             raise ValueError(f"top {top} of {experts} experts")
         if router_scores not in ("sigmoid", "softmax", "softmax_all") or weight_on not in ("input", "output"):
@@ -59,9 +64,13 @@ class MixtureOfExperts:
         if self.identity < 0 or count <= 0 or total % count or not 0 < keep <= count or keep * (total // count) < top:
             raise ValueError(f"{count} groups (keep {keep}) over {experts} + {self.identity} experts, top {top}")
         # the kernel that scores all experts serves every router that needs more than the largest logits
-        self.full_router = router_scores == "softmax_all" or self.correction or count > 1 or self.identity > 0
+        self.router_scale, self.act_consts, self.shared_gate = float(router_scale), act_consts, shared_gate
+        self.full_router = router_scores == "softmax_all" or self.correction or count > 1 or self.identity > 0 \
+            or self.router_scale != 1.0 or shared_gate is not None
         if self.full_router and router_scores == "softmax":
-            raise ValueError("a softmax over the chosen experts has no correction, groups or identity experts")
+            raise ValueError("a softmax over the chosen experts has no correction, groups, identity experts, scale or shared gate")
+        if shared_gate is not None and shared is None:
+            raise ValueError("a gate on the shared unit needs a shared unit")
         if self.identity and weight_on == "input":
             raise ValueError("identity experts weigh their output")
         if len(names) != (3 if gated else 2):
@@ -81,7 +90,7 @@ class MixtureOfExperts:
     def param_specs(cls, hidden_size, experts, top, expert_size, shared: Optional[PartSpec] = None,
                     router_name: str = "router", expert_prefix: str = "e", names=("gate", "up", "down"),
                     gated: bool = True, correction: bool = False, correction_name: str = "correction", identity: int = 0,
-                    **_) -> Dict[str, ParamSpec]:
+                    shared_gate: Optional[str] = None, **_) -> Dict[str, ParamSpec]:
         specs = {router_name: ParamSpec((experts + identity, hidden_size))}
         if correction:
             specs[correction_name] = ParamSpec((experts + identity,), "small")
@@ -93,10 +102,15 @@ class MixtureOfExperts:
         if shared is not None:
             for k, v in lookup("feed_forward", shared.kind).param_specs(**shared.params).items():
                 specs[shared.prefix + k] = v
+            if shared_gate is not None:
+                specs[shared.prefix + shared_gate] = ParamSpec((1, hidden_size))
         return specs
 
     def load(self, t: Dict[str, torch.Tensor]) -> None:
         self.w_router = t[self.router_name].contiguous()
+        if self.shared_gate is not None:
+            t = dict(t)
+            self.w_router = torch.cat([self.w_router, t.pop(self.shared_spec.prefix + self.shared_gate)], dim=0).contiguous()
         if self.correction:
             self.w_correction = t[self.correction_name].to(torch.float32).contiguous()
         if self.shared is not None:
@@ -130,7 +144,8 @@ class MixtureOfExperts:
         z = ops.linear(x, self.w_router, out_dtype=torch.float32)
         if self.full_router:
             ids, weights = ops.moe_route_grouped(z, self.top, "sigmoid" if self.router_scores == "sigmoid" else "softmax",
-                                                 self.w_correction, *self.groups)
+                                                 self.w_correction, *self.groups, scale=self.router_scale,
+                                                 experts=self.experts + self.identity)
         else:
             ids, weights = ops.moe_route(z, self.top, softmax_weights=self.router_scores == "softmax")
         rows = ids.numel()
@@ -142,8 +157,9 @@ class MixtureOfExperts:
         on_input = self.weight_on == "input"
         act = ops.moe_grouped(x, w_first, plan, self.top, gated=self.gated, gather=True,
                               weights=weights if on_input else None, act=self.activation,
-                              interleaved=self.interleaved, unary=not self.gated)
+                              interleaved=self.interleaved, unary=not self.gated, consts=self.act_consts)
         y = ops.moe_grouped(act, self.w_down, plan, self.top, gated=False, gather=False)
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
         return ops.moe_combine(y, plan, self.top, shared, self.dtype, weights=None if on_input else weights,
-                               identity_input=x if self.identity else None)
+                               identity_input=x if self.identity else None,
+                               shared_gate=None if self.shared_gate is None else z[:, self.experts + self.identity])
