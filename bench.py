@@ -1408,6 +1408,253 @@ def pevolorn_bench(args) -> int:
     return 0
 
 
+VIGONEX_SIZES = {
+    # width; residual streams; layers in the order delta rule (dense feed-forward), attention, attention, delta rule
+    # (mixtures), repeated; attention: heads, key/value heads, width of one map's queries and keys, value width (two maps
+    # of 64 cost what one of 128 does); delta rule: heads, width, rank; the mixture: experts, top, expert and shared widths
+    # (top * expert + shared = the dense width)
+    "1b": dict(width=2048, streams=2, layers=8, vocab=32768, a_heads=16, a_kv=4, a_dim=64, a_vdim=128, d_heads=16, d_dim=128,
+               rank=64, experts=32, top=4, expert_ff=1024, shared_ff=2048, ff=6144),
+    "8b": dict(width=4096, streams=2, layers=4, vocab=32768, a_heads=32, a_kv=8, a_dim=64, a_vdim=128, d_heads=32, d_dim=128,
+               rank=128, experts=64, top=4, expert_ff=2048, shared_ff=4096, ff=12288),
+}
+
+
+def _vigonex_at(z):
+    from tiny_llm_infer_b200.config.vigonex import (DenseConfig, DifferentialConfig, GeneralDeltaConfig, MixtureConfig,
+                                                     VigonexConfig, VigonexLayerConfig)
+    moe = MixtureConfig(z["expert_ff"], 7.0, z["experts"], z["top"], 2.5, z["shared_ff"], 7.0)
+    att = DifferentialConfig(z["a_heads"], z["a_kv"], z["a_dim"], z["a_vdim"], z["a_dim"] ** -0.5, 0.5, 50.0, 0.2, 1024)
+    delta = GeneralDeltaConfig(z["d_heads"], z["d_dim"], z["rank"])
+    kinds = [("general_delta", delta, DenseConfig(z["ff"])), ("attention", att, moe), ("attention", att, moe),
+             ("general_delta", delta, moe)]
+    return VigonexConfig(vocab=z["vocab"], width=z["width"], streams=z["streams"], norm_eps=1e-6, embedding_scale=2.0,
+                         logit_scale=0.5, layers=tuple(VigonexLayerConfig(*kinds[i % 4]) for i in range(z["layers"])))
+
+
+def vigonex_bench(args) -> int:
+    """``--design vigonex``: prefill and decode throughput of the Vigonex design at sizes that resemble a real model's
+    layers (random weights, bfloat16; two residual streams; layers in the order delta rule, attention with two maps
+    twice, delta rule; the first with a dense feed-forward, the others with mixtures), beside the closest models the
+    engine has at equal width, layers, feed-forward share and vocabulary, through the same step function: Panolorn
+    (capped attention, gated experts on every second layer) and Kaketar (three delta-rule layers in four, dense).  Then
+    the design's kernels one by one beside their relatives, with their share of the measured peaks.  One JSON line."""
+    import torch
+    from tiny_llm_infer_b200 import ops
+    from tiny_llm_infer_b200.config.panolorn import (AttentionMixerConfig, FeedForwardConfig, PanolornConfig,
+                                                      PanolornLayerConfig)
+    from tiny_llm_infer_b200.engine.batch import StepContext
+    from tiny_llm_infer_b200.parts.registry import lookup
+    from tiny_llm_infer_b200.parts.spec import PartSpec
+
+    hx = _DesignHarness(args)
+    device, pk, clocks, windows = hx.device, hx.pk, hx.clocks, hx.windows
+    tokens_pf, batch, context, steps, warmup = hx.tokens_pf, hx.batch, hx.context, hx.steps, hx.warmup
+    timed, run_model = hx.timed, hx.run_model
+    record = {"sizes": {}}
+    for size_name in ([args.model] if args.model in VIGONEX_SIZES else sorted(VIGONEX_SIZES)):
+        z = VIGONEX_SIZES[size_name]
+        L, W, H, G, D = z["layers"], z["width"], z["a_heads"], z["a_kv"], z["a_vdim"]
+        vcfg, kcfg = _vigonex_at(z), _kaketar_at(KAKETAR_SIZES[size_name])
+        pz = DESIGN_SIZES[size_name]
+        pcfg = PanolornConfig(vocab=z["vocab"], width=W, embedding_scale=math.sqrt(W), norm_eps=1e-5, layers=tuple(
+            PanolornLayerConfig("attention", AttentionMixerConfig(H, G, D, D, 1.0 / math.sqrt(D), 50.0, pz["chunk"]),
+                                FeedForwardConfig("dense", z["ff"]) if i % 2 == 0 else
+                                FeedForwardConfig("moe", pz["expert_ff"], experts=pz["experts"], top=pz["top"], shared_ff=pz["shared_ff"]))
+            for i in range(L)))
+        # every matrix of the model, and of a mixture the experts a token meets, or the ones a decode step of `batch`
+        # rows reads at most
+        v_all, v_kv, v_state = _model_costs(vcfg, context)
+        mixtures = sum(1 for i in range(L) if i % 4)
+        expert = 3 * W * z["expert_ff"]
+        v_params = {"active": v_all - mixtures * (z["experts"] - z["top"]) * expert,
+                    "read": v_all - mixtures * (z["experts"] - min(z["experts"], batch * z["top"])) * expert}
+        p_all, p_kv, _ = _model_costs(pcfg, context)
+        p_expert = 3 * W * pz["expert_ff"]
+        p_params = {"active": p_all - (L // 2) * (pz["experts"] - pz["top"]) * p_expert,
+                    "read": p_all - (L // 2) * (pz["experts"] - min(pz["experts"], batch * pz["top"])) * p_expert}
+        k_all, k_kv, k_state = _model_costs(kcfg, context)
+        entry = {"config": z, "params": {}}
+        for label, cfg, params, kvb, st in (("vigonex", vcfg, v_params, v_kv, v_state), ("panolorn", pcfg, p_params, p_kv, 0.0),
+                                            ("kaketar", kcfg, {"active": k_all, "read": k_all}, k_kv, k_state)):
+            print(f"[bench] design sizes {size_name}: {label}", file=sys.stderr, flush=True)
+            r = run_model(cfg, f"{label} {size_name}", params, kvb, st)
+            r["prefill_frac_of_measured"] = round(r["prefill_tflops"] / pk["bf16_tflops"], 4)
+            r["decode_hbm_frac_of_measured"] = round(r["decode_gbs"] / pk["hbm_gbs"], 4)
+            print(f"[bench] {r}", file=sys.stderr, flush=True)
+            entry[label] = r
+            entry["params"][label] = params
+        record["sizes"][size_name] = entry
+
+    # ---- kernels one by one at the larger sizes (L2 flushed between runs)
+    z = VIGONEX_SIZES["8b"]
+    W, S, bf, T = z["width"], z["streams"], torch.bfloat16, tokens_pf
+    kern = {}
+
+    def hbm(nbytes, ms):
+        return {"us": round(ms * 1e3, 1), "gbs": round(nbytes / ms / 1e6, 1), "frac_hbm": round(nbytes / ms / 1e6 / pk["hbm_gbs"], 3)}
+
+    def tensor(flops, ms):
+        return {"us": round(ms * 1e3, 1), "tflops": round(flops / ms / 1e9, 1), "frac_tensor": round(flops / ms / 1e9 / pk["bf16_tflops"], 3)}
+
+    # between two sub-layers: update of the streams with a gate, read, norm (and shift), beside the sums with a norm
+    n = 4 * T
+    x = torch.randn(n, S * W, device=device)
+    h = torch.randn(n, W, device=device)
+    delta, gate = (torch.randn(n, W, device=device).to(bf) for _ in range(2))
+    gain32, gain16 = torch.ones(W, device=device), torch.ones(W, device=device, dtype=bf)
+    bias, shift = torch.randn(W, device=device), torch.rand(W, device=device)
+    w_in, w_out, mix = torch.rand(S, device=device), torch.rand(S, device=device), torch.rand(S, S, device=device)
+    tail = torch.zeros(64, W, device=device)
+    one = torch.zeros(n, dtype=torch.int32, device=device)
+    seg = torch.tensor([[0, 0, n, 0]], dtype=torch.int32, device=device)
+    out = torch.empty_like(delta)
+    per = n * W
+
+    def read(shifted, rows=n, **more):
+        if shifted:
+            more.update(shift=shift, tail=tail, token_slot=one[:rows], seg_info=seg)
+        return ops.stream_read(x[:rows], S, gain32, 1e-6, bf, w_in=w_in, delta=delta[:rows], mix=mix, w_out=w_out, gate=gate[:rows],
+                               gate_bias=bias, delta_bias=bias, **more)
+    kern["stream_read_2_streams_gate"] = hbm(per * (8 * S + 2 + 2 + 2), timed(lambda: read(False)))
+    kern["stream_read_2_streams_gate_shift"] = hbm(per * (8 * S + 2 + 2 + 2 + 2), timed(lambda: read(True)))
+    kern["postnorm_add_rmsnorm"] = hbm(per * (8 + 2 + 2), timed(lambda: ops.add_rmsnorm(h, delta, gain16, 1e-5, out, post_gain=gain16, post_eps=1e-5)))
+    kern["add_rmsnorm"] = hbm(per * (8 + 2 + 2), timed(lambda: ops.add_rmsnorm(h, delta, gain16, 1e-5, out)))
+    few = torch.arange(64, dtype=torch.int32, device=device)
+    kern["stream_read_2_streams_gate_shift_64_single_tokens"] = {"us": round(timed(lambda: ops.stream_read(
+        x[:64], S, gain32, 1e-6, bf, w_in=w_in, delta=delta[:64], mix=mix, w_out=w_out, gate=gate[:64], gate_bias=bias, delta_bias=bias,
+        shift=shift, tail=tail, token_slot=few, single_tokens=True)) * 1e3, 1)}
+    kern["add_rmsnorm_64_rows"] = {"us": round(timed(lambda: ops.add_rmsnorm(h[:64], delta[:64], gain16, 1e-5, out[:64])) * 1e3, 1)}
+    # the start: embedding with sinusoids into every stream, beside the embedding with a learned position table
+    ids = torch.randint(0, 32768, (n,), device=device, dtype=torch.int32)
+    pos = torch.arange(n, device=device, dtype=torch.int32)
+    emb, ptab = torch.randn(32768, W, device=device).to(bf), torch.randn(n, W, device=device).to(bf)
+    freq = torch.rand(W // 2, 2, device=device) * torch.tensor([1.0, 1e-9], device=device)
+    kern["embedding_sinusoid_2_streams"] = hbm(per * (2 + 4 * S), timed(lambda: ops.embedding_sinusoid(ids, pos, emb, freq, 2.0, S)))
+    kern["kaketar_embedding_positions"] = hbm(per * (2 + 2 + 4), timed(lambda: ops.embedding_norm(ids, emb, h, 2.0, pos, ptab)))
+    del x, h, delta, gate, out, emb, ptab
+
+    rows, page, ctx_len = 64, 16, context
+
+    def context_for(segs):
+        seg, tiles, dec, row = [], [], [], 0
+        for s, (slot, p0, n) in enumerate(segs):
+            seg.append([slot, row, n, p0])
+            if n == 1:
+                dec.append(row)
+            else:
+                tiles += [(s, off) for off in range(0, n, 64)]
+            row += n
+        tiles.sort(key=lambda t: (t[1] % 256 != 0, t[1] % 128 != 0))
+        pos = torch.tensor([p0 + i for _, p0, n in segs for i in range(n)], dtype=torch.int32, device=device)
+        slot = torch.tensor([sl for sl, _, n in segs for _ in range(n)], dtype=torch.int32, device=device)
+        return StepContext(tokens=row, token_ids=None, positions=pos, token_slot=slot, want_rows=None, segments=[],
+                           seg_info=torch.tensor(seg, dtype=torch.int32, device=device),
+                           dec_rows=None if len(dec) == row else torch.tensor(dec, dtype=torch.int32, device=device),
+                           n_dec=len(dec), pf_tiles=torch.tensor(tiles, dtype=torch.int32, device=device).view(-1, 2),
+                           n_tiles=len(tiles), n_tiles128=sum(1 for t in tiles if t[1] % 128 == 0),
+                           n_tiles256=sum(1 for t in tiles if t[1] % 256 == 0), max_context=ctx_len, max_segment=max(n for _, _, n in segs))
+
+    # attention with two maps of 64 per head over values of 128, beside Panolorn's capped attention of 128 (the same
+    # cache bytes; the same multiplications of queries with keys, twice those of weights with values)
+    H, G, d, D = z["a_heads"], z["a_kv"], z["a_dim"], z["a_vdim"]
+    n_pages = rows * ctx_len // page
+    table = torch.arange(n_pages, dtype=torch.int32, device=device).view(rows, ctx_len // page).contiguous()
+    pool = (torch.randn(n_pages, 2 * G * page * D, device=device) * 0.5).to(bf)
+    k_plane = pool[:, :G * page * D].unflatten(1, (G, page, D))
+    v_plane = pool[:, G * page * D:].unflatten(1, (G, page, D))
+    in_bias = torch.randn((H + 2 * G) * D, device=device)
+    slopes = torch.rand(H, device=device) * 0.01
+    for what, segs in (("prefill_2048", [(0, 0, T)]), ("decode_64_rows_ctx_2048", [(i, ctx_len - 1, 1) for i in range(rows)])):
+        ctx = context_for(segs)
+        n = ctx.tokens
+        q = torch.randn(n, H * D, device=device).to(bf)
+        o = torch.empty_like(q)
+        proj = torch.randn(n, (H + 2 * G) * D + H * D, device=device).to(bf)
+        full_gate = proj[:, (H + 2 * G) * D:]
+        moved = n * ((H + 2 * G) * D * 2 + (H + 2 * G) * D * 2)
+        kern[f"qkv_store_bias_temperature_{what}"] = hbm(moved, timed(lambda: ops.qkv_unit_store(
+            proj, q, ctx.positions, ctx.token_slot, table, k_plane, v_plane, page, H, G, D, D, None, bias=in_bias, q_temperature=(0.2, 1024))))
+        kern[f"panolorn_qkv_store_unit_{what}"] = hbm(moved, timed(lambda: ops.qkv_unit_store(
+            proj, q, ctx.positions, ctx.token_slot, table, k_plane, v_plane, page, H, G, D, D, 1e-6)))
+        runs = {"attention_two_maps_cap": (lambda: ops.attention_biased(
+                    q, k_plane, v_plane, ctx.positions, ctx.token_slot, table, page, H, G, d, D, d ** -0.5, o, softcap=50.0, ctx=ctx,
+                    difference=(0.4, 1e-6, 0.5)), 2.0 * H * 2 * (d + D)),
+                "panolorn_attention_cap_slopes_gate": (lambda: ops.attention_biased(
+                    q, k_plane, v_plane, ctx.positions, ctx.token_slot, table, page, H, G, D, D, D ** -0.5, o, softcap=50.0,
+                    chunk=4096, sink=True, slopes=slopes, gate=full_gate, ctx=ctx), 2.0 * H * 2 * D)}
+        for name, (fn, flops) in runs.items():
+            ms = timed(fn)
+            kern[f"{name}_{what}"] = tensor(flops * T * (T + 1) / 2, ms) if what.startswith("prefill") else \
+                hbm(rows * ctx_len * 2 * G * D * 2, ms)
+    del pool, k_plane, v_plane
+
+    # the delta rule with a removal rate per channel beside Kaketar's with one write strength, at equal state: 2048
+    # tokens of one request, and 64 one-token rows (state read and written once per row)
+    Hd, dd = z["d_heads"], z["d_dim"]
+    inner = Hd * dd
+    words = ops.delta_rule_state_floats(Hd, Hd, dd, dd, 1)
+
+    def scan_record(n, ms, io, work):
+        total = io + work + (0 if n == T else 2 * rows * words * 4)
+        return {"us": round(ms * 1e3, 1), "tokens_per_s": round(n / ms * 1e3, 1), "gbs": round(total / ms / 1e6, 1),
+                "frac_hbm": round(total / ms / 1e6 / pk["hbm_gbs"], 3)}
+
+    for what, n, seg in (("prefill_2048", T, [[0, 0, T, 0]]), ("decode_64_rows", rows, None)):
+        slots = torch.zeros(n, dtype=torch.int32, device=device) if seg else torch.arange(n, dtype=torch.int32, device=device)
+        seg_info = torch.tensor(seg, dtype=torch.int32, device=device) if seg else None
+        state = torch.zeros(rows, words, device=device)
+        proj = torch.randn(n, 5 * inner, device=device).to(bf)
+        zz, zb, ab, w2 = torch.randn(n, inner, device=device), torch.randn(inner, device=device), torch.randn(inner, device=device), torch.ones(inner, device=device)
+        ms = timed(lambda: ops.erase_delta_rule(proj, 4 * inner, zz, zb, ab, math.exp(-0.5), proj[:, 3 * inner:4 * inner], "sigmoid", w2,
+                                                True, 1e-6, slots, seg_info, state, Hd, dd, dd, 1e-6, bf))
+        kern[f"erase_delta_rule_{what}"] = scan_record(n, ms, n * inner * (5 * 2 + 4 + 2), n * 6 * inner * 4 * 2)
+        del state
+        taps = 4
+        state = torch.zeros(rows, ops.delta_rule_state_floats(Hd, Hd, dd, dd, taps), device=device)
+        proj = torch.randn(n, 3 * inner + Hd, device=device).to(bf)
+        conv_w = (torch.randn(3 * inner, taps, device=device) * 0.5).to(bf)
+        conv_t, rate, w1 = conv_w.t().contiguous(), torch.ones(Hd, device=device), torch.ones(dd, device=device)
+        second = torch.randn(n, 2 * inner, device=device)
+        ms = timed(lambda: ops.delta_rule(proj, conv_w, taps, second[:, :inner], zb, rate, second[:, inner:], w1, 1e-6, slots, seg_info,
+                                          state, Hd, Hd, dd, dd, dd ** -0.5, 1e-6, bf, conv_t=conv_t))
+        kern[f"kaketar_delta_rule_{what}"] = scan_record(n, ms, n * inner * (3 * 2 + 2 * 4 + 2), n * 5 * inner * 4 * 2)
+        del state
+
+    # the mixture: clamped experts, a scaled router and a gated shared expert, beside Panolorn's (SiLU) at equal widths
+    E, top, eff, sff = z["experts"], z["top"], z["expert_ff"], z["shared_ff"]
+    zl = torch.randn(8192, E + 1, device=device)
+    kern["moe_route_scaled_8192_rows"] = {"us": round(timed(lambda: ops.moe_route_grouped(zl, top, "softmax", scale=2.5, experts=E)) * 1e3, 1)}
+    zl2 = zl[:, :E].contiguous()
+    kern["moe_route_8192_rows"] = {"us": round(timed(lambda: ops.moe_route(zl2, top)) * 1e3, 1)}
+    cls, names = lookup("feed_forward", "moe"), ("gate", "up", "down")
+    clamped = dict(activation="clamped_swish", act_consts=(7.0, 1.702))
+    kinds = {"mixture_clamped_gated_shared": dict(router_scores="softmax_all", router_scale=2.5, weight_on="output", shared_gate="sg", **clamped),
+             "panolorn_mixture": dict(activation="silu")}
+    for name, more in kinds.items():
+        act = {k: v for k, v in more.items() if k in ("activation", "act_consts")}
+        params = dict(hidden_size=W, experts=E, top=top, expert_size=eff, names=names,
+                      shared=PartSpec("swiglu", dict(hidden_size=W, intermediate_size=sff, names=names, **act), "shared."), **more)
+        part = cls(dtype=bf, device=device, **params)
+        part.load({k: (torch.randn(spec.shape, device=device) * 0.02).to(bf) for k, spec in cls.param_specs(**params).items()})
+        for n in (8, 8192):
+            xx = torch.randn(n, W, device=device).to(bf)
+            ms = timed(lambda: part.forward(xx, None))
+            kern[f"{name}_{n}_rows"] = hbm(3 * W * (min(E, n * top) * eff + sff) * 2, ms) if n == 8 else \
+                tensor(2.0 * n * 3 * W * (top * eff + sff), ms)
+        del part
+    ops.check_error_word(device)
+    record["kernels"] = kern
+    clock_record = clocks.stop(windows)
+    first = record["sizes"][sorted(record["sizes"])[0]]["vigonex"]
+    print(json.dumps({"metric": f"decode tok/s @ batch {batch} (Vigonex design sizes, context {context}, 1 B200)",
+                      "value": first["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": warmup,
+                      "ms_per_step": first["decode_ms"], "higher_is_better": True, "dtype": "bf16", "data": "synthetic",
+                      "design": "vigonex", "clocks": clock_record, "peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"]},
+                      **record}))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1415,7 +1662,7 @@ def main() -> int:
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--batch", type=int, default=8)
-    ap.add_argument("--model", default="8b", choices=sorted(set(MODELS) | set(DESIGN_SIZES) | set(TETODRA_SIZES) | set(PEVOLORN_SIZES)),
+    ap.add_argument("--model", default="8b", choices=sorted(set(MODELS) | set(DESIGN_SIZES) | set(TETODRA_SIZES) | set(PEVOLORN_SIZES) | set(VIGONEX_SIZES)),
                     help="the sizes: 8b is the benchmark configuration, 0.6b and 32b the other two the reference is quoted on")
     ap.add_argument("--layers", type=int, default=None,
                     help="fewer layers than the model has (named in the record) if memory or time needs it")
@@ -1428,7 +1675,7 @@ def main() -> int:
     ap.add_argument("--skip-check", action="store_true", help="leave out the logits check before the timed phases")
     ap.add_argument("--ref-all", action="store_true",
                     help="reference arm: its model_main --bench at batch 1, 8 and 64 instead of --batch alone")
-    ap.add_argument("--design", default=None, choices=["panolorn", "kaketar", "tetodra", "pevolorn"],
+    ap.add_argument("--design", default=None, choices=["panolorn", "kaketar", "tetodra", "pevolorn", "vigonex"],
                     help="instead of the default workload: this design's prefill and decode throughput at sizes that "
                          "resemble a real model's layers beside Qwen3 dense at equal sizes, and its kernels one by one")
     ap.add_argument("--only", default="all", choices=["all", "prefill", "decode", "e2e", "mixed", "p128"],
@@ -1438,7 +1685,8 @@ def main() -> int:
         if args.gpus != 1 or args.impl != "ours":
             print("bench.py: --design runs this engine on one GPU")
             return 2
-        return {"kaketar": kaketar_bench, "tetodra": tetodra_bench, "pevolorn": pevolorn_bench}.get(args.design, design_bench)(args)
+        return {"kaketar": kaketar_bench, "tetodra": tetodra_bench, "pevolorn": pevolorn_bench,
+                "vigonex": vigonex_bench}.get(args.design, design_bench)(args)
     if args.model not in MODELS:
         ap.error(f"--model {args.model} goes with --design")
     model_name, model_sizes = MODELS[args.model]

@@ -286,8 +286,8 @@ __global__ void stream_tails_kernel(const int* __restrict__ seg_info, const T* h
 // ---------------------------------------------------------------- embedding with sinusoids
 // out[t, s, :] = table[ids[t], :] * scale + position vector, the same for every stream s: column 2 i of the position
 // vector is sin(p f_i), column 2 i + 1 cos(p f_i).  A frequency comes as two floats (its rounded value and what the
-// rounding left): the product p f_i is formed with its own rounding error beside it, which is applied to the sine and
-// the cosine as a first-order correction, so that angles of many turns keep float32 accuracy.
+// rounding left): the product p f_i is formed with its own rounding error beside it, and sine and cosine are those of
+// the sum of the two (a few terms of the small one's series), so that angles of many turns keep float32 accuracy.
 template <typename TW>
 __global__ void embedding_sinusoid_kernel(const int* __restrict__ ids, const int* __restrict__ positions,
                                           const TW* __restrict__ table, const float2* __restrict__ freq, float scale,
@@ -308,8 +308,9 @@ __global__ void embedding_sinusoid_kernel(const int* __restrict__ ids, const int
             const float ang = p * f.x, rest = fmaf(p, f.y, fmaf(p, f.x, -ang));
             float sn, cs;
             sincosf(ang, &sn, &cs);
-            a = to_f32<TW>(src[2 * i]) * scale + (sn + rest * cs);
-            if (two) b = to_f32<TW>(src[2 * i + 1]) * scale + (cs - rest * sn);
+            const float c2 = 1.0f - 0.5f * rest * rest, s2 = rest * (1.0f - rest * rest * (1.0f / 6.0f));   // cos, sin of rest
+            a = to_f32<TW>(src[2 * i]) * scale + fmaf(sn, c2, cs * s2);
+            if (two) b = to_f32<TW>(src[2 * i + 1]) * scale + fmaf(cs, c2, -sn * s2);
         }
         for (int s = 0; s < streams; ++s) {
             dst[(size_t)s * width + 2 * i] = a;
