@@ -1428,7 +1428,7 @@ def _vigonex_at(z):
     delta = GeneralDeltaConfig(z["d_heads"], z["d_dim"], z["rank"])
     kinds = [("general_delta", delta, DenseConfig(z["ff"])), ("attention", att, moe), ("attention", att, moe),
              ("general_delta", delta, moe)]
-    return VigonexConfig(vocab=z["vocab"], width=z["width"], streams=z["streams"], norm_eps=1e-6, embedding_scale=2.0,
+    return VigonexConfig(vocab=z["vocab"], width=z["width"], streams=z["streams"], norm_eps=1e-6, embedding_scale=50.0,
                          logit_scale=0.5, layers=tuple(VigonexLayerConfig(*kinds[i % 4]) for i in range(z["layers"])))
 
 

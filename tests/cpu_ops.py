@@ -48,13 +48,18 @@ def _act(g, act):
     return g / (1 + torch.exp(-g))
 
 
-def swiglu(gate_up, out, interleaved=False, act="silu"):
+def swiglu(gate_up, out, interleaved=False, act="silu", consts=None):
     inter = out.shape[1]
     if interleaved:                  # groups of sixteen columns: eight gates, their eight ups
         pairs = gate_up.float().reshape(gate_up.shape[0], inter // 8, 2, 8)
         g, u = pairs[:, :, 0].reshape(-1, inter), pairs[:, :, 1].reshape(-1, inter)
     else:
         g, u = gate_up[:, :inter].float(), gate_up[:, inter:].float()
+    if act == "clamped_swish":
+        limit, slope = consts
+        g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+        out.copy_((g * torch.sigmoid(slope * g) * (u + 1.0)).to(out.dtype))
+        return out
     out.copy_((_act(g, act) * u).to(out.dtype))
     return out
 
@@ -77,10 +82,10 @@ def interleave_gate_up(gate, up):
     return torch.stack([gate.reshape(inter // 8, 8, k), up.reshape(inter // 8, 8, k)], dim=1).reshape(2 * inter, k)
 
 
-def linear_swiglu(x, w_gate_up, out_dtype, interleaved=False, act="silu"):
+def linear_swiglu(x, w_gate_up, out_dtype, interleaved=False, act="silu", consts=None):
     gate_up = linear(x, w_gate_up, out_dtype)
     out = torch.empty((x.shape[0], w_gate_up.shape[0] // 2), dtype=out_dtype)
-    return swiglu(gate_up, out, interleaved, act)
+    return swiglu(gate_up, out, interleaved, act, consts)
 
 
 def qk_norm_rope_store(qkv, q_gain, k_gain, eps, inv_freq, rotary_dim, positions, token_slot,

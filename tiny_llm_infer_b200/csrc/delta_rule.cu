@@ -262,7 +262,9 @@ struct ScanLayout {
     }
 };
 
-// R lanes share a column, each keeps PER rows of it at most.  The chunks of tokens come through two stages
+// R lanes share a column, each keeps PER rows of it at most.  A thread takes NC neighbouring columns (one, or two in
+// steps of long portions): it reads a token's rows from shared memory once for all of them, and those reads are what a
+// long portion's time goes with.  A column's arithmetic is the same either way.  The chunks of tokens come through two stages
 // filled by cp.async, so that the next chunk is on its way while this one is walked.  A token's step, per
 // thread: S <- g S, dot = sum S k, u = beta (v - dot), S <- S + k u, o = sum S q.  Only S is carried from token
 // to token; the read-out's sum is off that path.
@@ -280,8 +282,8 @@ struct ScanLayout {
 enum ScanMode : int { kScanDelta = 0, kScanPlain = 1, kScanMemory = 2, kScanHeadDecay = 3, kScanErase = 4 };
 __host__ __device__ constexpr int scan_vecs(int mode) { return mode == kScanErase ? 4 : 3; }
 
-template <int R, int PER, int MODE>
-__global__ void __launch_bounds__(256, 2)
+template <int R, int PER, int MODE, int NC>
+__global__ void __launch_bounds__(NC == 1 ? 256 : 128, 2)
 delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ token_slot,
                   const float* qn, const float* kn, const float* vv, const float* decay,
                   const float* beta, float* state, long long state_stride, int heads,
@@ -302,9 +304,8 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
     }
     if (slot < 0 || len <= 0) return;
     const int per = (dk + R - 1) / R;
-    const int r = threadIdx.x % R, jl = threadIdx.x / R;       // lane of the column, column of the block
+    const int r = threadIdx.x % R, jl = threadIdx.x / R * NC;  // lane of the columns, the first of them in the block
     const int j = col0 + jl;
-    const bool live = j < dv;
     const int kvh = head / (heads / kv_heads);
     const int stage_floats = L::stage_floats(cols);
     float* o_s = sm + 2 * stage_floats;               // [chunk][cols]
@@ -362,15 +363,19 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
     issue(0, 0);
     // in the request's state the element (row r * per + il, column j) lies at [il][j][r]: a warp reads whole lines
     float* st_ptr = state + (long long)slot * state_stride + (size_t)head * per * dv * R;
-    float2 S2[PER / 2];                               // rows il = 2 p and 2 p + 1 of this lane
-#pragma unroll
-    for (int il = 0; il < PER; il += 2) {
-        S2[il >> 1].x = (live && il < per) ? st_ptr[((size_t)il * dv + j) * R + r] : 0.0f;
-        S2[il >> 1].y = (live && il + 1 < per) ? st_ptr[((size_t)(il + 1) * dv + j) * R + r] : 0.0f;
-    }
-
+    float2 S2[NC][PER / 2];                           // rows il = 2 p and 2 p + 1 of this lane
     float* top_ptr = state + (long long)slot * state_stride + aux_off + (size_t)head * dv + j;
-    float top = (MODE == kScanMemory && live) ? *top_ptr : 0.0f;      // running maximum of the gates' logarithms
+    float top[NC];                                    // running maximum of the gates' logarithms
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+        const bool live = j + c < dv;
+#pragma unroll
+        for (int il = 0; il < PER; il += 2) {
+            S2[c][il >> 1].x = (live && il < per) ? st_ptr[((size_t)il * dv + j + c) * R + r] : 0.0f;
+            S2[c][il >> 1].y = (live && il + 1 < per) ? st_ptr[((size_t)(il + 1) * dv + j + c) * R + r] : 0.0f;
+        }
+        top[c] = (MODE == kScanMemory && live) ? top_ptr[c] : 0.0f;
+    }
     const bool has_beta = beta != nullptr;
     int stage = 0;
     for (int c0 = 0; c0 < len; c0 += kScanChunk, stage ^= 1) {
@@ -392,98 +397,120 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
         // every thread walks the tokens (the shuffles want whole warps); one without a column carries zeros
         // two rows at a time with the packed float32 instructions of sm_100 (each half rounds as the scalar
         // instruction would): Sg = S g, dot += Sg k, S = Sg + k u, o += S q: four instructions for two rows
-        auto step = [&](int tt) -> float {
+        auto step = [&](int tt, float (&o)[NC]) {
             const float4* kr = reinterpret_cast<const float4*>(k_s + tt * L::kRow + r * kLane);
             const float4* qr = reinterpret_cast<const float4*>(q_s + tt * L::kRow + r * kLane);
             const float4* gr = reinterpret_cast<const float4*>(g_s + tt * L::kRow + r * kLane);
             const float4* er = reinterpret_cast<const float4*>(e_s + tt * L::kRow + r * kLane);
             float2 kk[PER / 2];
-            float2 dot_a = make_float2(0.0f, 0.0f), dot_b = dot_a;
-            float write = 1.0f;
-            float2 keep2 = make_float2(1.0f, 1.0f);
-            if (MODE == kScanMemory) {
-                const float fi = f_s[tt], ii = b_s[tt];
-                const float top_new = fmaxf(fi + top, ii);
-                const float keep = expf(fi + top - top_new);
-                write = expf(ii - top_new);
-                top = top_new;
-                keep2 = make_float2(keep, keep);
-            } else if (MODE == kScanPlain) {
-                write = has_beta ? b_s[tt] : 1.0f;
-            } else if (MODE == kScanHeadDecay) {
-                keep2 = make_float2(b_s[tt], b_s[tt]);
-                write = f_s[tt];
+            float2 dot_a[NC], dot_b[NC], keep2[NC];
+            float write[NC];
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+                dot_a[c] = dot_b[c] = make_float2(0.0f, 0.0f);
+                write[c] = 1.0f;
+                keep2[c] = make_float2(1.0f, 1.0f);
+                if (MODE == kScanMemory) {
+                    const float fi = f_s[tt], ii = b_s[tt];
+                    const float top_new = fmaxf(fi + top[c], ii);
+                    const float keep = expf(fi + top[c] - top_new);
+                    write[c] = expf(ii - top_new);
+                    top[c] = top_new;
+                    keep2[c] = make_float2(keep, keep);
+                } else if (MODE == kScanPlain) {
+                    write[c] = has_beta ? b_s[tt] : 1.0f;
+                } else if (MODE == kScanHeadDecay) {
+                    keep2[c] = make_float2(b_s[tt], b_s[tt]);
+                    write[c] = f_s[tt];
+                }
             }
 #pragma unroll
             for (int il = 0; il < PER; il += 4) {
                 const float4 k4 = kr[il >> 2];
                 kk[il >> 1] = make_float2(k4.x, k4.y);
                 kk[(il >> 1) + 1] = make_float2(k4.z, k4.w);
-                if (MODE == kScanErase) {                 // the removal reads the state before its decay
-                    dot_a = __ffma2_rn(S2[il >> 1], kk[il >> 1], dot_a);
-                    dot_b = __ffma2_rn(S2[(il >> 1) + 1], kk[(il >> 1) + 1], dot_b);
+                float4 g4 = make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+                if (kDecayRows) g4 = gr[il >> 2];
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    float2& s0 = S2[c][il >> 1];
+                    float2& s1 = S2[c][(il >> 1) + 1];
+                    if (MODE == kScanErase) {                 // the removal reads the state before its decay
+                        dot_a[c] = __ffma2_rn(s0, kk[il >> 1], dot_a[c]);
+                        dot_b[c] = __ffma2_rn(s1, kk[(il >> 1) + 1], dot_b[c]);
+                    }
+                    s0 = __fmul2_rn(s0, kDecayRows ? make_float2(g4.x, g4.y) : keep2[c]);
+                    s1 = __fmul2_rn(s1, kDecayRows ? make_float2(g4.z, g4.w) : keep2[c]);
+                    if (MODE == kScanDelta) {
+                        dot_a[c] = __ffma2_rn(s0, kk[il >> 1], dot_a[c]);
+                        dot_b[c] = __ffma2_rn(s1, kk[(il >> 1) + 1], dot_b[c]);
+                    }
                 }
-                if (MODE == kScanMemory || MODE == kScanHeadDecay) {
-                    S2[il >> 1] = __fmul2_rn(S2[il >> 1], keep2);
-                    S2[(il >> 1) + 1] = __fmul2_rn(S2[(il >> 1) + 1], keep2);
+            }
+            float2 u2[NC], gone[NC], o_a[NC], o_b[NC];
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+                float u;
+                if (MODE == kScanErase) {
+                    const float2 dsum = __fadd2_rn(dot_a[c], dot_b[c]);
+                    const float dot = -lanes_sum<R>(dsum.x + dsum.y);
+                    gone[c] = make_float2(dot, dot);
+                    u = v_s[tt * cols + jl + c];
+                } else if (MODE == kScanDelta) {
+                    const float2 dsum = __fadd2_rn(dot_a[c], dot_b[c]);
+                    const float dot = lanes_sum<R>(dsum.x + dsum.y);
+                    u = b_s[tt] * (v_s[tt * cols + jl + c] - dot);
                 } else {
-                    const float4 g4 = gr[il >> 2];
-                    S2[il >> 1] = __fmul2_rn(S2[il >> 1], make_float2(g4.x, g4.y));
-                    S2[(il >> 1) + 1] = __fmul2_rn(S2[(il >> 1) + 1], make_float2(g4.z, g4.w));
+                    u = write[c] * v_s[tt * cols + jl + c];
                 }
-                if (MODE == kScanDelta) {
-                    dot_a = __ffma2_rn(S2[il >> 1], kk[il >> 1], dot_a);
-                    dot_b = __ffma2_rn(S2[(il >> 1) + 1], kk[(il >> 1) + 1], dot_b);
-                }
+                u2[c] = make_float2(u, u);
+                o_a[c] = o_b[c] = make_float2(0.0f, 0.0f);
             }
-            float u;
-            float2 gone = make_float2(0.0f, 0.0f);
-            if (MODE == kScanErase) {
-                const float2 dsum = __fadd2_rn(dot_a, dot_b);
-                const float dot = -lanes_sum<R>(dsum.x + dsum.y);
-                gone = make_float2(dot, dot);
-                u = v_s[tt * cols + jl];
-            } else if (MODE == kScanDelta) {
-                const float2 dsum = __fadd2_rn(dot_a, dot_b);
-                const float dot = lanes_sum<R>(dsum.x + dsum.y);
-                u = b_s[tt] * (v_s[tt * cols + jl] - dot);
-            } else {
-                u = write * v_s[tt * cols + jl];
-            }
-            const float2 u2 = make_float2(u, u);
-            float2 o_a = make_float2(0.0f, 0.0f), o_b = o_a;
 #pragma unroll
             for (int il = 0; il < PER; il += 4) {
                 const float4 q4 = qr[il >> 2];
-                if (MODE == kScanErase) {
-                    const float4 e4 = er[il >> 2];
-                    S2[il >> 1] = __ffma2_rn(make_float2(e4.x, e4.y), gone, S2[il >> 1]);
-                    S2[(il >> 1) + 1] = __ffma2_rn(make_float2(e4.z, e4.w), gone, S2[(il >> 1) + 1]);
+                float4 e4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                if (MODE == kScanErase) e4 = er[il >> 2];
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    float2& s0 = S2[c][il >> 1];
+                    float2& s1 = S2[c][(il >> 1) + 1];
+                    if (MODE == kScanErase) {
+                        s0 = __ffma2_rn(make_float2(e4.x, e4.y), gone[c], s0);
+                        s1 = __ffma2_rn(make_float2(e4.z, e4.w), gone[c], s1);
+                    }
+                    s0 = __ffma2_rn(kk[il >> 1], u2[c], s0);
+                    s1 = __ffma2_rn(kk[(il >> 1) + 1], u2[c], s1);
+                    o_a[c] = __ffma2_rn(s0, make_float2(q4.x, q4.y), o_a[c]);
+                    o_b[c] = __ffma2_rn(s1, make_float2(q4.z, q4.w), o_b[c]);
                 }
-                S2[il >> 1] = __ffma2_rn(kk[il >> 1], u2, S2[il >> 1]);
-                S2[(il >> 1) + 1] = __ffma2_rn(kk[(il >> 1) + 1], u2, S2[(il >> 1) + 1]);
-                o_a = __ffma2_rn(S2[il >> 1], make_float2(q4.x, q4.y), o_a);
-                o_b = __ffma2_rn(S2[(il >> 1) + 1], make_float2(q4.z, q4.w), o_b);
             }
-            const float2 osum = __fadd2_rn(o_a, o_b);
-            const float o = lanes_sum<R>(osum.x + osum.y);
-            if (MODE == kScanMemory && j == dv - 1) return fmaxf(fabsf(o), expf(-top)) + floor_eps;
-            return o;
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+                const float2 osum = __fadd2_rn(o_a[c], o_b[c]);
+                o[c] = lanes_sum<R>(osum.x + osum.y);
+                if (MODE == kScanMemory && j + c == dv - 1) o[c] = fmaxf(fabsf(o[c]), expf(-top[c])) + floor_eps;
+            }
         };
         if (n == kScanChunk) {
             // a whole chunk: unrolled, the read-outs kept in registers until the end, so that no store to shared
             // memory stands between a token's loads and the next one's and they can be issued ahead
-            float o_reg[kScanChunk];
+            float o_reg[kScanChunk][NC];
 #pragma unroll
-            for (int tt = 0; tt < kScanChunk; ++tt) o_reg[tt] = step(tt);
+            for (int tt = 0; tt < kScanChunk; ++tt) step(tt, o_reg[tt]);
             if (r == 0) {
 #pragma unroll
-                for (int tt = 0; tt < kScanChunk; ++tt) o_s[tt * cols + jl] = o_reg[tt];
+                for (int tt = 0; tt < kScanChunk; ++tt)
+#pragma unroll
+                    for (int c = 0; c < NC; ++c) o_s[tt * cols + jl + c] = o_reg[tt][c];
             }
         } else {
             for (int tt = 0; tt < n; ++tt) {
-                const float oq = step(tt);
-                if (r == 0) o_s[tt * cols + jl] = oq;
+                float oq[NC];
+                step(tt, oq);
+                if (r == 0)
+#pragma unroll
+                    for (int c = 0; c < NC; ++c) o_s[tt * cols + jl + c] = oq[c];
             }
         }
         __syncthreads();
@@ -498,12 +525,14 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
             }
         }
     }
-    if (MODE == kScanMemory && live && r == 0) *top_ptr = top;
-    if (live) {
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+        if (j + c >= dv) continue;
+        if (MODE == kScanMemory && r == 0) top_ptr[c] = top[c];
 #pragma unroll
         for (int il = 0; il < PER; il += 2) {
-            if (il < per) st_ptr[((size_t)il * dv + j) * R + r] = S2[il >> 1].x;
-            if (il + 1 < per) st_ptr[((size_t)(il + 1) * dv + j) * R + r] = S2[il >> 1].y;
+            if (il < per) st_ptr[((size_t)il * dv + j + c) * R + r] = S2[c][il >> 1].x;
+            if (il + 1 < per) st_ptr[((size_t)(il + 1) * dv + j + c) * R + r] = S2[c][il >> 1].y;
         }
     }
 }
@@ -910,7 +939,8 @@ int tllm_delta_prepare(const void* proj, int ld, int dtype, const void* conv_w, 
 }
 
 // seg_info: int[segments][4] = slot, first row, length, first position; null: every row is a portion of one token.
-int tllm_delta_scan(const int* seg_info, int segments, const int* token_slot, const float* qn, const float* kn,
+// rows: rows of the step (how long the portions are on average decides how many columns a thread takes).
+int tllm_delta_scan(const int* seg_info, int segments, int rows, const int* token_slot, const float* qn, const float* kn,
                     const float* vv, const float* decay, const float* beta, float* state, long long state_stride,
                     int heads, int kv_heads, int dk, int dv, float* o_raw, int mode, const float* fgate,
                     const float* erase, long long aux_off, float floor_eps, float* den, cudaStream_t stream) {
@@ -930,12 +960,14 @@ int tllm_delta_scan(const int* seg_info, int segments, const int* token_slot, co
     // multiprocessor in all where the value width allows it (a column does not depend on the others, so the
     // result is the same however they are dealt)
     int cols = 256 / r;
-    const int min_cols = 32 / r > 1 ? 32 / r : 1;
+    const bool two = r < 32 && per > 8;               // sizes whose rows are worth reading for two columns at once
+    const int nc = two && seg_info != nullptr && rows >= 16LL * segments ? 2 : 1;
+    const int min_cols = nc * (32 / r > 1 ? 32 / r : 1);
     const int sms = sm_count_cached() > 0 ? sm_count_cached() : 148;
     while (cols > min_cols && cols / 2 >= dv) cols /= 2;
-    while (cols > min_cols && (long long)segments * heads * ((dv + cols - 1) / cols) < sms) cols /= 2;
+    while (cols > min_cols && (long long)segments * heads * ((dv + cols - 1) / cols) < (nc == 2 ? sms * 3 / 4 : sms)) cols /= 2;
     const int col_blocks = (dv + cols - 1) / cols;
-    const int threads = cols * r;
+    const int threads = cols / nc * r;
     TLLM_REQUIRE(col_blocks <= 65535, "delta_scan: sizes %d x %d do not fit", dk, dv);
     const auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; };
     const int vec = dk % 4 == 0 && per % 4 == 0 && aligned(qn) && aligned(kn) && (decay == nullptr || aligned(decay)) &&
@@ -950,15 +982,20 @@ int tllm_delta_scan(const int* seg_info, int segments, const int* token_slot, co
     } while (0)
 #define SCAN_MODE(RR, PP, MM)                                                                                           \
     do {                                                                                                         \
+        if (nc == 2) SCAN_NC(RR, PP, MM, (RR < 32 && PP == 16 ? 2 : 1));                                         \
+        else SCAN_NC(RR, PP, MM, 1);                                                                             \
+    } while (0)
+#define SCAN_NC(RR, PP, MM, NN)                                                                                  \
+    do {                                                                                                         \
         const size_t smem = ((size_t)2 * ScanLayout<RR, PP, scan_vecs(MM)>::stage_floats(cols) + (size_t)scan_chunk(RR) * cols) * sizeof(float); \
         TLLM_REQUIRE(smem <= 200 * 1024, "delta_scan: sizes %d x %d do not fit", dk, dv);                         \
         static OncePerDevice configured;                                                                         \
         if (configured.first()) {                                                                                \
-            cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<RR, PP, MM>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
+            cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<RR, PP, MM, NN>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
             if (e != cudaSuccess) { set_error("delta_scan: %s", cudaGetErrorString(e)); return (int)e; }         \
             configured.done();                                                                                   \
         }                                                                                                        \
-        launch_pdl(kPdlOther, delta_scan_kernel<RR, PP, MM>, dim3(segments, heads, col_blocks), dim3(threads), smem, stream, \
+        launch_pdl(kPdlOther, delta_scan_kernel<RR, PP, MM, NN>, dim3(segments, heads, col_blocks), dim3(threads), smem, stream, \
                    seg_info, token_slot, qn, kn, vv, decay, beta, state, state_stride, heads, kv_heads, dk, dv,  \
                    cols, vec, o_raw, fgate, erase, aux_off, floor_eps, den);                                            \
     } while (0)
@@ -970,6 +1007,7 @@ int tllm_delta_scan(const int* seg_info, int segments, const int* token_slot, co
     else SCAN(32, 16);
 #undef SCAN
 #undef SCAN_MODE
+#undef SCAN_NC
     return finish_launch("delta_scan");
 }
 

@@ -80,7 +80,7 @@ def _declare(h) -> None:
         "tllm_activation": [vp, vp, i32, i32, i32, i32, vp, vp, i32, i32, i32, vp],
         "tllm_delta_prepare": [vp, i32, i32, vp, vp, i32, vp, i32, vp, vp, vp, vp, i64, i32, i32, i32, i32, f32, f32,
                                vp, vp, vp, vp, vp, i32, i32, i32, vp],
-        "tllm_delta_scan": [vp, i32, vp, vp, vp, vp, vp, vp, vp, i64, i32, i32, i32, i32, vp, i32, vp, vp, i64, f32, vp, vp],
+        "tllm_delta_scan": [vp, i32, i32, vp, vp, vp, vp, vp, vp, vp, i64, i32, i32, i32, i32, vp, i32, vp, vp, i64, f32, vp, vp],
         "tllm_erase_prepare": [vp, i32, i32, i32, vp, i32, vp, vp, f32, vp, i32, i32, i32, f32, vp, vp, vp, vp, vp, i32, vp],
         "tllm_stream_read": [vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, f32, vp, i32, vp, vp, vp, i64, i32, vp, vp, i32, i32, i32, vp],
         "tllm_stream_tails": [vp, i32, vp, i32, vp, i64, i32, vp],
@@ -1031,7 +1031,7 @@ def delta_rule(proj: torch.Tensor, conv_w: torch.Tensor, taps: int, a: torch.Ten
                                     int(decay_per_head), -1 if beta_col is None else int(beta_col), _stream()),
            "delta_prepare")
     segments = tokens if seg_info is None else seg_info.shape[0]
-    _check(lib().tllm_delta_scan(_p(seg_info), segments, _p(token_slot), _p(qn), _p(kn), _p(vv), _p(decay), _p(beta),
+    _check(lib().tllm_delta_scan(_p(seg_info), segments, tokens, _p(token_slot), _p(qn), _p(kn), _p(vv), _p(decay), _p(beta),
                                  _p(state), state.stride(0), heads, kv_heads, dk, dv, _p(o_raw), SCAN_DELTA, None, None, 0, 0.0,
                                  None, _stream()), "delta_scan")
     return _delta_finish(o_raw, gate, out_weight, False, eps, token_slot, tokens, heads, kv_heads, dk, dv, out_dtype,
@@ -1068,7 +1068,7 @@ def erase_delta_rule(proj: torch.Tensor, a_col: int, z: torch.Tensor, z_bias: to
                                     _p(token_slot), heads, dk, dv, float(unit_eps), _p(qn), _p(kn), _p(vv), _p(decay),
                                     _p(erase), tokens, _stream()), "erase_prepare")
     segments = tokens if seg_info is None else seg_info.shape[0]
-    _check(lib().tllm_delta_scan(_p(seg_info), segments, _p(token_slot), _p(qn), _p(kn), _p(vv), _p(decay), None,
+    _check(lib().tllm_delta_scan(_p(seg_info), segments, tokens, _p(token_slot), _p(qn), _p(kn), _p(vv), _p(decay), None,
                                  _p(state), state.stride(0), heads, heads, dk, dv, _p(o_raw), SCAN_ERASE, None, _p(erase), 0,
                                  0.0, None, _stream()), "delta_scan")
     return _delta_finish(o_raw, gate, out_weight, weight_per_head, eps, token_slot, tokens, heads, heads, dk, dv,
@@ -1127,7 +1127,7 @@ def linear_recurrence(proj: torch.Tensor, kind: str, z: torch.Tensor, z_bias: to
                                      _p(decay), _p(wgate), _p(fgate), tokens, _stream()), "linear_prepare")
     segments = tokens if seg_info is None else seg_info.shape[0]
     aux_off = delta_rule_state_floats(heads, heads, dk, cols, 1) if memory else 0
-    _check(lib().tllm_delta_scan(_p(seg_info), segments, _p(token_slot), _p(qn), _p(kn), _p(vv), _p(decay), _p(wgate),
+    _check(lib().tllm_delta_scan(_p(seg_info), segments, tokens, _p(token_slot), _p(qn), _p(kn), _p(vv), _p(decay), _p(wgate),
                                  _p(state), state.stride(0), heads, heads, dk, cols, _p(o_raw),
                                  SCAN_MEMORY if memory else SCAN_PLAIN, _p(fgate), None, aux_off, float(floor_eps), _p(den),
                                  _stream()), "delta_scan")
@@ -1177,7 +1177,7 @@ def state_space(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: Optional[torch
                                   _p(token_slot), _p(state), state.stride(0), tail_off, heads, groups, n_state, head_dim,
                                   _p(qn), _p(kn), _p(vv), _p(decay), _p(step), tokens, _stream()), "ssd_prepare")
     segments = tokens if seg_info is None else seg_info.shape[0]
-    _check(lib().tllm_delta_scan(_p(seg_info), segments, _p(token_slot), _p(qn), _p(kn), _p(vv), None, _p(decay),
+    _check(lib().tllm_delta_scan(_p(seg_info), segments, tokens, _p(token_slot), _p(qn), _p(kn), _p(vv), None, _p(decay),
                                  _p(state), state.stride(0), heads, groups, n_state, head_dim, _p(o_raw), SCAN_HEAD_DECAY,
                                  _p(step), None, 0, 0.0, None, _stream()), "delta_scan")
     out = torch.empty((tokens, inner), dtype=out_dtype, device=proj.device)

@@ -110,7 +110,10 @@ class MixtureOfExperts:
         self.w_router = t[self.router_name].contiguous()
         if self.shared_gate is not None:
             t = dict(t)
-            self.w_router = torch.cat([self.w_router, t.pop(self.shared_spec.prefix + self.shared_gate)], dim=0).contiguous()
+            rows = [self.w_router, t.pop(self.shared_spec.prefix + self.shared_gate)]
+            pad = -sum(r.shape[0] for r in rows) % 8            # rows of the product stay whole 16-byte pieces
+            rows.append(torch.zeros((pad, self.hidden), dtype=rows[0].dtype, device=rows[0].device))
+            self.w_router = torch.cat(rows, dim=0).contiguous()
         if self.correction:
             self.w_correction = t[self.correction_name].to(torch.float32).contiguous()
         if self.shared is not None:
