@@ -281,7 +281,8 @@ def test_two_maps_over_a_long_request_with_shared_out_keys(case):
 # ----------------------------------------------------------------------------- the delta rule with a removal rate per channel
 ERASE_CASES = [dict(H=4, d=16, rank=8), dict(H=3, d=10, rank=5), dict(H=2, d=128, rank=24), dict(H=1, d=72, rank=16),
                dict(H=5, d=64, rank=8), dict(H=2, d=200, rank=3), dict(H=1, d=264, rank=8), dict(H=7, d=1, rank=2),
-               dict(H=6, d=32, dv=56, rank=8), dict(H=2, d=20, dv=6, rank=4)]
+               dict(H=6, d=32, dv=56, rank=8), dict(H=2, d=20, dv=6, rank=4),
+               dict(H=10, d=128, rank=8), dict(H=21, d=60, rank=8), dict(H=8, d=200, rank=4)]     # two columns per thread
 
 
 @pytest.mark.parametrize("case", ERASE_CASES, ids=lambda c: f"h{c['H']}d{c['d']}v{c.get('dv', c['d'])}r{c['rank']}")
@@ -329,6 +330,53 @@ def test_delta_rule_with_removal_per_channel(case, dtype):
     if d == 1:                     # a head of one number is normed to its sign: a read-out near zero may fall either way
         limit = 1e-3 if dtype == torch.float32 else 2.0
     assert whole < limit and cutup < limit, (whole, cutup)
+
+
+@pytest.mark.parametrize("dk,dv", [(64, 96), (128, 64), (250, 40)])
+@pytest.mark.parametrize("mode", ["delta", "channel_decay", "log_gates", "state_space", "erase"])
+def test_scan_with_two_columns_per_thread_changes_nothing(mode, dk, dv):
+    """Every recurrence of the scan kernel: portions of 48 tokens (two columns per thread at these sizes) against the same
+    tokens in portions of 8 (one), bit for bit, states included."""
+    from tiny_llm_infer_b200 import ops
+    H, slots, L = 3552 // (3 * dv) + 4, 3, 48
+    torch.manual_seed(dk)
+    if mode == "state_space":
+        width, words = 2 * H * dv + 2 * H * dk + H, ops.state_space_state_floats(H, H, dk, dv, 1)
+    elif mode == "erase":
+        width, words = 3 * H * dk + 2 * H * dv, ops.delta_rule_state_floats(H, H, dk, dv, 1)
+    elif mode == "delta":
+        width, words = 2 * H * dk + H * dv + H, ops.delta_rule_state_floats(H, H, dk, dv, 1)
+    else:
+        width, words = H * (2 * dk + dv), ops.linear_recurrence_state_floats(mode, H, dk, dv)
+    proj = torch.randn(slots, L, -(-width // 8) * 8, device=DEV) * 0.3
+    z = torch.randn(slots, L, 2 * H if mode == "log_gates" else H * dk, device=DEV)
+    gate = torch.randn(slots, L, H * dv, device=DEV)
+    zb, ab, rate = torch.randn(z.shape[2], device=DEV), torch.randn(H * dk, device=DEV), torch.rand(H, device=DEV)
+    w1, wh, hb = torch.ones(dv, device=DEV), torch.ones(H * dv, device=DEV), torch.randn(H, device=DEV)
+    conv = torch.ones(2 * H * dk + H * dv, 1, device=DEV)
+
+    def run(step):
+        state = torch.zeros(slots, words, device=DEV)
+        outs = []
+        for p0 in range(0, L, step):
+            cut = [t[:, p0:p0 + step].reshape(slots * step, -1).contiguous() for t in (proj, z, gate)]
+            ctx = make_ctx([(i, p0, step) for i in range(slots)])
+            common = (ctx.token_slot, ctx.seg_info, state)
+            f32 = torch.float32
+            if mode == "erase":
+                o = ops.erase_delta_rule(cut[0], 2 * H * dk + 2 * H * dv, cut[1], zb, ab, 0.6, cut[2], "sigmoid", wh, True, 1e-6, *common,
+                                         H, dk, dv, 1e-6, f32)
+            elif mode == "delta":
+                o = ops.delta_rule(cut[0], conv, 1, cut[1], zb, rate, cut[2], w1, 1e-6, *common, H, H, dk, dv, 0.1, 1e-6, f32)
+            elif mode == "state_space":
+                o = ops.state_space(cut[0], conv, None, 1, hb, rate, hb, wh, 1e-6, 1, *common, H, H, dk, dv, f32)
+            else:
+                o = ops.linear_recurrence(cut[0], mode, cut[1], zb, 8.0, cut[2], "silu", w1, False, 1e-6, *common, H, dk, dv, 0.1, f32)
+            outs.append(o.view(slots, step, -1))
+        return torch.cat(outs, dim=1), state
+    (long, s1), (short, s2) = run(L), run(8)
+    assert torch.isfinite(long).all() and long.abs().max() > 0
+    assert torch.equal(long, short) and torch.equal(s1, s2)
 
 
 # ----------------------------------------------------------------------------- experts
