@@ -4,5 +4,6 @@ from .kaketar import KaketarConfig
 from .panolorn import PanolornConfig
 from .pevolorn import PevolornConfig
 from .qwen3 import Qwen3Config
+from .sozavik import SozavikConfig
 from .tetodra import TetodraConfig
 from .vigonex import VigonexConfig

@@ -74,6 +74,29 @@ __device__ __forceinline__ float mod_score(float dot, float slope, int dist, con
 }
 
 // ---------------------------------------------------------------- norm of q and k, write of k and v
+// How queries and keys are normed: not at all, every head by itself (gains of dk numbers, shared by the heads), or
+// all heads of a token together, the queries as one vector and the keys as another (gains of q_heads * dk and
+// kv_heads * dk numbers).
+enum QkNorm : int { kQkNone = 0, kQkPerHead = 1, kQkWhole = 2 };
+
+// Values mixed with another layer's values of the same token, v <- keep v + share (first + first_bias), before they
+// are written: `first` points at the token-0 row of those values as they were projected (heads side by side), `stride`
+// elements from one token to the next.  Null: the values as they are.
+template <typename T>
+struct ValueMix {
+    const T* first;
+    int stride;
+    const float* bias;
+    float keep, share;
+};
+
+// Sums of squares of a token's queries and of its keys, each over all heads (every thread gets both).
+template <typename F>
+__device__ __forceinline__ void whole_sums(F square_sum, int q_len, int k_len, float* scratch, float& q_sum, float& k_sum) {
+    q_sum = block_sum(square_sum(0, q_len), scratch);
+    k_sum = block_sum(square_sum(q_len, q_len + k_len), scratch);
+}
+
 // proj[t] = q heads | k heads | v heads | (anything else).  One warp per head of a token.
 template <typename T>
 __global__ void qkv_unit_store_kernel(const T* proj, int row_stride, const T* __restrict__ q_gain,
@@ -82,8 +105,9 @@ __global__ void qkv_unit_store_kernel(const T* proj, int row_stride, const T* __
                                       const int* __restrict__ block_table, int max_pages, int page_size,
                                       T* k_plane, T* v_plane, long long page_stride, T* q_out,
                                       int q_heads, int kv_heads, int dk, int dv, int store,
-                                      const float* __restrict__ inv_freq, int rot_dims, float temp_coef,
-                                      int temp_every, int v_from_k, const float* __restrict__ bias) {
+                                      const float* __restrict__ inv_freq, int rot_dims, int pairs, float temp_coef,
+                                      int temp_every, int v_from_k, const float* __restrict__ bias, ValueMix<T> mix) {
+    __shared__ float scratch[32];
     TLLM_PDL_ENTER();
     const int t = blockIdx.x;
     const int slot = token_slot[t];
@@ -102,18 +126,32 @@ __global__ void qkv_unit_store_kernel(const T* proj, int row_stride, const T* __
         if (page < 0) store = 0;          // no page held: nothing to write (the host reserves before a step)
     }
     const int total = q_heads + 2 * kv_heads;
+    float q_whole = 1.0f, k_whole = 1.0f;
+    if (do_norm == kQkWhole) {
+        whole_sums([&](int from, int to) {
+            float sum = 0.0f;
+            for (int c = from + threadIdx.x; c < to; c += blockDim.x) { const float x = at(c); sum += x * x; }
+            return sum;
+        }, q_heads * dk, kv_heads * dk, scratch, q_whole, k_whole);
+        q_whole = 1.0f / sqrtf(q_whole / (float)(q_heads * dk) + eps);
+        k_whole = 1.0f / sqrtf(k_whole / (float)(kv_heads * dk) + eps);
+    }
     for (int head = warp; head < total; head += warps) {
         if (head < q_heads + kv_heads) {
             const bool is_q = head < q_heads;
             const size_t src = (size_t)head * dk;
             const T* gain = is_q ? q_gain : k_gain;
-            float sum = 0.0f;
-            for (int e = lane; e < dk; e += 32) {
-                const float x = at(src + e);
-                sum += x * x;
+            if (do_norm == kQkWhole && gain != nullptr) gain += (size_t)(is_q ? head : head - q_heads) * dk;
+            float sc = is_q ? q_whole : k_whole;
+            if (do_norm == kQkPerHead) {
+                float sum = 0.0f;
+                for (int e = lane; e < dk; e += 32) {
+                    const float x = at(src + e);
+                    sum += x * x;
+                }
+                sum = warp_sum(sum);
+                sc = 1.0f / sqrtf(sum / (float)dk + eps);
             }
-            sum = warp_sum(sum);
-            const float sc = do_norm ? 1.0f / sqrtf(sum / (float)dk + eps) : 1.0f;
             T* dst;
             if (is_q) dst = q_out + ((size_t)t * q_heads + head) * dk;
             else if (store) dst = k_plane + page_base + ((size_t)(head - q_heads) * page_size + in_page) * dk;
@@ -124,13 +162,14 @@ __global__ void qkv_unit_store_kernel(const T* proj, int row_stride, const T* __
             for (int e = lane; e < dk; e += 32) {
                 float x = at(src + e) * sc;
                 if (gain != nullptr && do_norm) x *= to_f32<T>(gain[e]);
-                if (e < rot_dims) {               // element e turns with its partner half a rotated width away
-                    const int partner = e < half ? e + half : e - half;
+                if (e < rot_dims) {               // element e turns with its neighbour, or with its partner half a rotated width away
+                    const bool low = pairs ? (e & 1) == 0 : e < half;
+                    const int partner = pairs ? e ^ 1 : (low ? e + half : e - half);
                     float y = at(src + partner) * sc;
                     if (gain != nullptr && do_norm) y *= to_f32<T>(gain[partner]);
-                    const float ang = (float)pos * inv_freq[e < half ? e : e - half];
+                    const float ang = (float)pos * inv_freq[pairs ? e >> 1 : (low ? e : e - half)];
                     const float c = cosf(ang), sn = sinf(ang);
-                    x = e < half ? x * c - y * sn : x * c + y * sn;
+                    x = low ? x * c - y * sn : x * c + y * sn;
                 }
                 dst[e] = from_f32<T>(x * temp);
             }
@@ -140,7 +179,13 @@ __global__ void qkv_unit_store_kernel(const T* proj, int row_stride, const T* __
             const size_t src = v_from_k ? (size_t)(q_heads + g) * dk
                                         : (size_t)(q_heads + kv_heads) * dk + (size_t)g * dv;
             T* dst = v_plane + page_base + ((size_t)g * page_size + in_page) * dv;
-            if (bias != nullptr) for (int e = lane; e < dv; e += 32) dst[e] = from_f32<T>(at(src + e));
+            if (mix.first != nullptr) {
+                const T* other = mix.first + (size_t)t * mix.stride + (size_t)g * dv;
+                for (int e = lane; e < dv; e += 32) {
+                    const float f = to_f32<T>(other[e]) + (mix.bias != nullptr ? mix.bias[(size_t)g * dv + e] : 0.0f);
+                    dst[e] = from_f32<T>(mix.keep * at(src + e) + mix.share * f);
+                }
+            } else if (bias != nullptr) for (int e = lane; e < dv; e += 32) dst[e] = from_f32<T>(at(src + e));
             else for (int e = lane; e < dv; e += 32) dst[e] = row[src + e];
         }
     }
@@ -149,8 +194,8 @@ __global__ void qkv_unit_store_kernel(const T* proj, int row_stride, const T* __
 // The same for bfloat16 rows whose widths are multiples of eight: a group of GS lanes (a power of two; dk / 8 of
 // them at work) holds a head, eight elements to a lane, so a warp takes 32 / GS heads at once with 16-byte
 // loads and stores.  The token's cosines and sines are made once, in shared memory, for all its heads; the
-// partner of a rotated element sits half / 8 lanes away (half a multiple of eight).  The arithmetic per
-// element is that of the kernel above.
+// partner of a rotated element sits half / 8 lanes away (half a multiple of eight) or, turning in neighbouring
+// pairs, in the same lane.  The arithmetic per element is that of the kernel above.
 __device__ __forceinline__ void load8(const bf16* p, float (&v)[8]) {
     const uint4 raw = *reinterpret_cast<const uint4*>(p);
     const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
@@ -169,9 +214,10 @@ qkv_unit_store_vec_kernel(const bf16* proj, int row_stride, const bf16* __restri
                           const int* __restrict__ positions, const int* __restrict__ token_slot,
                           const int* __restrict__ block_table, int max_pages, int page_size, bf16* k_plane,
                           bf16* v_plane, long long page_stride, bf16* q_out, int q_heads, int kv_heads, int dk,
-                          int dv, int store, const float* __restrict__ inv_freq, int rot_dims, float temp_coef,
-                          int temp_every, int v_from_k, const float* __restrict__ bias) {
+                          int dv, int store, const float* __restrict__ inv_freq, int rot_dims, int pairs, float temp_coef,
+                          int temp_every, int v_from_k, const float* __restrict__ bias, ValueMix<bf16> mix) {
     extern __shared__ float cos_sin[];                      // cos of the token's `half` angles, then their sines
+    __shared__ float scratch[32];
     TLLM_PDL_ENTER();
     const int t = blockIdx.x;
     const int slot = token_slot[t];
@@ -198,27 +244,48 @@ qkv_unit_store_vec_kernel(const bf16* proj, int row_stride, const bf16* __restri
     const int grp = lane / GS, gl = lane % GS, e0 = gl * 8;
     const int normed = q_heads + kv_heads;
     const float q_temp = temp_every > 0 ? 1.0f + temp_coef * logf((float)((pos + 1) / temp_every) + 1.0f) : 1.0f;
+    // eight columns of the row as the kernel sees them: the projection plus its bias, if it has one, in float32
+    auto at8 = [&](size_t c, float (&v)[8]) {
+        load8(row + c, v);
+        if (bias != nullptr) {
+            const float4 b0 = *reinterpret_cast<const float4*>(bias + c);
+            const float4 b1 = *reinterpret_cast<const float4*>(bias + c + 4);
+            v[0] += b0.x; v[1] += b0.y; v[2] += b0.z; v[3] += b0.w;
+            v[4] += b1.x; v[5] += b1.y; v[6] += b1.z; v[7] += b1.w;
+        }
+    };
+    float q_whole = 1.0f, k_whole = 1.0f;
+    if (do_norm == kQkWhole) {
+        whole_sums([&](int from, int to) {
+            float sum = 0.0f;
+            for (int c = from + threadIdx.x * 8; c < to; c += blockDim.x * 8) {
+                float v[8];
+                at8(c, v);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) sum += v[e] * v[e];
+            }
+            return sum;
+        }, q_heads * dk, kv_heads * dk, scratch, q_whole, k_whole);
+        q_whole = 1.0f / sqrtf(q_whole / (float)(q_heads * dk) + eps);
+        k_whole = 1.0f / sqrtf(k_whole / (float)(kv_heads * dk) + eps);
+    }
     for (int base = warp * kPerWarp; base < normed; base += warps * kPerWarp) {
         const int head = base + grp;
         const bool is_q = head < q_heads;
         const bool active = head < normed && e0 < dk;
         float v[8] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
-        if (active) {
-            load8(row + (size_t)head * dk + e0, v);
-            if (bias != nullptr) {                           // the projection's bias, added in float32
-                const float4 b0 = *reinterpret_cast<const float4*>(bias + (size_t)head * dk + e0);
-                const float4 b1 = *reinterpret_cast<const float4*>(bias + (size_t)head * dk + e0 + 4);
-                v[0] += b0.x; v[1] += b0.y; v[2] += b0.z; v[3] += b0.w;
-                v[4] += b1.x; v[5] += b1.y; v[6] += b1.z; v[7] += b1.w;
-            }
+        if (active) at8((size_t)head * dk + e0, v);
+        float sc = is_q ? q_whole : k_whole;
+        if (do_norm == kQkPerHead) {
+            float sum = 0.0f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) sum += v[e] * v[e];
+#pragma unroll
+            for (int o = GS / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            sc = 1.0f / sqrtf(sum / (float)dk + eps);
         }
-        float sum = 0.0f;
-#pragma unroll
-        for (int e = 0; e < 8; ++e) sum += v[e] * v[e];
-#pragma unroll
-        for (int o = GS / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-        const float sc = do_norm ? 1.0f / sqrtf(sum / (float)dk + eps) : 1.0f;
         const bf16* gain = is_q ? q_gain : k_gain;
+        if (do_norm == kQkWhole && gain != nullptr) gain += (size_t)(is_q ? head : head - q_heads) * dk;
         if (active && gain != nullptr && do_norm) {
             float gn[8];
             load8(gain + e0, gn);
@@ -228,7 +295,17 @@ qkv_unit_store_vec_kernel(const bf16* proj, int row_stride, const bf16* __restri
 #pragma unroll
             for (int e = 0; e < 8; ++e) v[e] *= sc;
         }
-        if (half > 0) {                                      // every lane takes part in the exchange
+        if (pairs) {
+#pragma unroll
+            for (int e = 0; e < 8; e += 2) {
+                if (e0 + e < rot_dims) {
+                    const int i = (e0 + e) >> 1;
+                    const float c = cos_sin[i], sn = cos_sin[half + i], x = v[e], y = v[e + 1];
+                    v[e] = x * c - y * sn;
+                    v[e + 1] = y * c + x * sn;
+                }
+            }
+        } else if (half > 0) {                               // every lane takes part in the exchange
             const bool turns = e0 < rot_dims, low = e0 < half;
             const int from = turns ? (low ? lane + half / 8 : lane - half / 8) : lane;
             const int i0 = low ? e0 : e0 - half;
@@ -260,17 +337,23 @@ qkv_unit_store_vec_kernel(const bf16* proj, int row_stride, const bf16* __restri
         for (int c = threadIdx.x; c < kv_heads * per_head; c += blockDim.x) {
             const int g = c / per_head, j = c - g * per_head;
             bf16* dst = v_plane + page_base + ((size_t)g * page_size + in_page) * dv + j * 8;
-            if (bias == nullptr) {
+            if (bias == nullptr && mix.first == nullptr) {
                 *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(src0 + (size_t)g * dv + j * 8);
                 continue;
             }
             float v[8];
-            load8(src0 + (size_t)g * dv + j * 8, v);
-            const float* b = bias + (src0 - row) + (size_t)g * dv + j * 8;
+            at8((src0 - row) + (size_t)g * dv + j * 8, v);
+            if (mix.first != nullptr) {
+                float f[8];
+                load8(mix.first + (size_t)t * mix.stride + (size_t)g * dv + j * 8, f);
+                const float* b = mix.bias != nullptr ? mix.bias + (size_t)g * dv + j * 8 : nullptr;
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v[e] = mix.keep * v[e] + mix.share * (f[e] + (b != nullptr ? b[e] : 0.0f));
+            }
             uint4 raw;
             __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&raw);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) h2[e] = __floats2bfloat162_rn(v[2 * e] + b[2 * e], v[2 * e + 1] + b[2 * e + 1]);
+            for (int e = 0; e < 4; ++e) h2[e] = __floats2bfloat162_rn(v[2 * e], v[2 * e + 1]);
             *reinterpret_cast<uint4*>(dst) = raw;
         }
     }
@@ -1151,15 +1234,18 @@ int tllm_qkv_unit_store(const void* proj, int row_stride, const void* q_gain, co
                         int do_norm, const int* positions, const int* token_slot, const int* block_table,
                         int max_pages, int page_size, void* k_plane, void* v_plane, long long page_stride,
                         void* q_out, int dtype, int tokens, int q_heads, int kv_heads, int dk, int dv,
-                        int store, const float* inv_freq, int rot_dims, float temp_coef, int temp_every, int v_from_k,
-                        const float* bias, cudaStream_t stream) {
+                        int store, const float* inv_freq, int rot_dims, int rot_pairs, float temp_coef, int temp_every,
+                        int v_from_k, const float* bias, const void* mix_first, int mix_stride, const float* mix_bias,
+                        float mix_share, cudaStream_t stream) {
     TLLM_REQUIRE(tokens >= 0 && q_heads > 0 && kv_heads > 0 && dk > 0 && dv > 0, "qkv_unit_store: bad sizes");
     TLLM_REQUIRE(row_stride >= (q_heads + kv_heads) * dk + (v_from_k ? 0 : kv_heads * dv), "qkv_unit_store: rows of %d are too short", row_stride);
     TLLM_REQUIRE(rot_dims >= 0 && rot_dims <= dk && rot_dims % 2 == 0 && (rot_dims == 0 || inv_freq != nullptr),
                  "qkv_unit_store: a rotation of %d of %d elements", rot_dims, dk);
     TLLM_REQUIRE(!v_from_k || dv == dk, "qkv_unit_store: keys of width %d cannot serve as values of width %d", dk, dv);
     TLLM_REQUIRE(temp_every >= 0, "qkv_unit_store: negative constant");
+    TLLM_REQUIRE(do_norm >= kQkNone && do_norm <= kQkWhole, "qkv_unit_store: unknown norm %d", do_norm);
     TLLM_REQUIRE(!do_norm || eps > 0.0f, "qkv_unit_store: eps must be positive");
+    TLLM_REQUIRE(mix_first == nullptr || (!v_from_k && mix_stride >= kv_heads * dv), "qkv_unit_store: other values in rows of %d", mix_stride);
     TLLM_REQUIRE(!store || (k_plane && v_plane && block_table && page_size > 0 && max_pages > 0),
                  "qkv_unit_store: no cache to write to");
     TLLM_REQUIRE(q_out != nullptr, "qkv_unit_store: no place for the queries");
@@ -1170,17 +1256,19 @@ int tllm_qkv_unit_store(const void* proj, int row_stride, const void* q_gain, co
     launch_pdl(kPdlQk, qkv_unit_store_kernel<T>, dim3(tokens), dim3(warps * 32), 0, stream, (const T*)proj,   \
                row_stride, (const T*)q_gain, (const T*)k_gain, eps, do_norm, positions, token_slot,           \
                block_table, max_pages, page_size, (T*)k_plane, (T*)v_plane, page_stride, (T*)q_out, q_heads,  \
-               kv_heads, dk, dv, store, inv_freq, rot_dims, temp_coef, temp_every, v_from_k, bias)
+               kv_heads, dk, dv, store, inv_freq, rot_dims, rot_pairs, temp_coef, temp_every, v_from_k, bias, \
+               ValueMix<T>{(const T*)mix_first, mix_stride, mix_bias, 1.0f - mix_share, mix_share})
     auto aligned16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; };
-    const bool vec = dtype == kBF16 && dk % 8 == 0 && dv % 8 == 0 && dk <= 256 && rot_dims % 16 == 0 &&
+    const bool vec = dtype == kBF16 && dk % 8 == 0 && dv % 8 == 0 && dk <= 256 && (rot_pairs || rot_dims % 16 == 0) &&
                      row_stride % 8 == 0 && page_stride % 8 == 0 && aligned16(proj) && aligned16(q_out) &&
-                     aligned16(k_plane) && aligned16(v_plane) && aligned16(q_gain) && aligned16(k_gain) && aligned16(bias);
+                     aligned16(k_plane) && aligned16(v_plane) && aligned16(q_gain) && aligned16(k_gain) && aligned16(bias) &&
+                     (mix_first == nullptr || (aligned16(mix_first) && mix_stride % 8 == 0));
 #define STORE_VEC(GS)                                                                                             \
     launch_pdl(kPdlQk, qkv_unit_store_vec_kernel<GS>, dim3(tokens), dim3(256), (size_t)rot_dims * sizeof(float),  \
                stream, (const bf16*)proj, row_stride, (const bf16*)q_gain, (const bf16*)k_gain, eps, do_norm,     \
                positions, token_slot, block_table, max_pages, page_size, (bf16*)k_plane, (bf16*)v_plane,          \
-               page_stride, (bf16*)q_out, q_heads, kv_heads, dk, dv, store, inv_freq, rot_dims, temp_coef,        \
-               temp_every, v_from_k, bias)
+               page_stride, (bf16*)q_out, q_heads, kv_heads, dk, dv, store, inv_freq, rot_dims, rot_pairs, temp_coef, \
+               temp_every, v_from_k, bias, ValueMix<bf16>{(const bf16*)mix_first, mix_stride, mix_bias, 1.0f - mix_share, mix_share})
     if (vec) {
         if (dk <= 8) STORE_VEC(1);
         else if (dk <= 16) STORE_VEC(2);

@@ -24,13 +24,18 @@ template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __f
 
 // Activation of the gate in a gated feed-forward unit, act(gate) * up, by code.
 // kActClampedSwish belongs to gated units only: it bounds gate and up before they meet (`gated_unit`).
-// kActTanh belongs to plain products only.
-enum GateAct : int { kActSilu = 0, kActGeluTanh = 1, kActGeluErf = 2, kActRelu2 = 3, kActClampedSwish = 4, kActTanh = 5 };
+// kActTanh belongs to plain products only, kActRelu to gated units.
+enum GateAct : int { kActSilu = 0, kActGeluTanh = 1, kActGeluErf = 2, kActRelu2 = 3, kActClampedSwish = 4, kActTanh = 5, kActRelu = 6 };
 
 // Constants of a gated unit whose activation has some (kActClampedSwish).
 struct GateConst {
     float limit, slope;
 };
+
+// Whether a gated unit knows the activation (the clamped swish with its constant).
+inline bool gated_act_ok(int act, float limit) {
+    return act == kActSilu || act == kActGeluTanh || act == kActRelu || (act == kActClampedSwish && limit > 0.0f);
+}
 
 __device__ __forceinline__ float gate_act(float g, int act) {
     if (act == kActGeluTanh)   // 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3)))
@@ -42,6 +47,7 @@ __device__ __forceinline__ float gate_act(float g, int act) {
         return r * r;
     }
     if (act == kActTanh) return tanhf(g);
+    if (act == kActRelu) return fmaxf(g, 0.0f);
     return g / (1.0f + expf(-g));
 }
 

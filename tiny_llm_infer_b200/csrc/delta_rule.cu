@@ -278,8 +278,9 @@ struct ScanLayout {
 // (token, head) for all rows of S and a write strength likewise, S <- a S + k (w v)^T; the decays come in `beta`
 // [., heads], the strengths in `fgate` [., heads], and `decay` is not read.  kScanErase: a delta rule whose removal has
 // a rate per key channel and reads the state before its decay, S <- g S - e (k^T S)^T + k v^T with k the unit key and
-// e = rate * k in `erase` (v comes already multiplied by the key's length); no beta.
-enum ScanMode : int { kScanDelta = 0, kScanPlain = 1, kScanMemory = 2, kScanHeadDecay = 3, kScanErase = 4 };
+// e = rate * k in `erase` (v comes already multiplied by the key's length); no beta.  kScanFixedDecay: no correction, and one
+// decay per head that no token changes, S <- a_h S + k v^T, the a_h in `fgate` [heads]; neither `decay` nor `beta` are read.
+enum ScanMode : int { kScanDelta = 0, kScanPlain = 1, kScanMemory = 2, kScanHeadDecay = 3, kScanErase = 4, kScanFixedDecay = 5 };
 __host__ __device__ constexpr int scan_vecs(int mode) { return mode == kScanErase ? 4 : 3; }
 
 template <int R, int PER, int MODE, int NC>
@@ -377,6 +378,7 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
         top[c] = (MODE == kScanMemory && live) ? top_ptr[c] : 0.0f;
     }
     const bool has_beta = beta != nullptr;
+    const float fixed = MODE == kScanFixedDecay ? fgate[head] : 1.0f;
     int stage = 0;
     for (int c0 = 0; c0 < len; c0 += kScanChunk, stage ^= 1) {
         const int n = min(kScanChunk, len - c0);
@@ -422,6 +424,8 @@ delta_scan_kernel(const int* __restrict__ seg_info, const int* __restrict__ toke
                 } else if (MODE == kScanHeadDecay) {
                     keep2[c] = make_float2(b_s[tt], b_s[tt]);
                     write[c] = f_s[tt];
+                } else if (MODE == kScanFixedDecay) {
+                    keep2[c] = make_float2(fixed, fixed);
                 }
             }
 #pragma unroll
@@ -663,8 +667,12 @@ __global__ void delta_finish_vec_kernel(const float* o_raw, const TG* gate, int 
 //                        exp(inv_tau * logsigmoid(z));
 //   kLinearLogGates      z [T, 2 heads] float32 + bias = write logits | keep logits, each capped as cap tanh(. / cap);
 //                        the write's logarithm is the capped logit, the keep's is logsigmoid of its capped logit; the
-//                        values get one more column of ones (the normaliser of a matrix memory), vv is [T, heads, dv + 1].
-enum LinearKind : int { kLinearChannelDecay = 0, kLinearLogGates = 1 };
+//                        values get one more column of ones (the normaliser of a matrix memory), vv is [T, heads, dv + 1];
+//   kLinearFixedDecay    no gates: the decays are the heads' own constants, which the scan reads itself.
+// act: 0 q, k and v as projected, 1 SiLU of each (in float32, before q's scale).
+enum LinearKind : int { kLinearChannelDecay = 0, kLinearLogGates = 1, kLinearFixedDecay = 2 };
+
+__device__ __forceinline__ float linear_input(float x, int act) { return act == 1 ? x / (1.0f + expf(-x)) : x; }
 
 __device__ __forceinline__ float log_sigmoid_f32(float z) {
     return fminf(z, 0.0f) - log1pf(expf(-fabsf(z)));
@@ -672,7 +680,7 @@ __device__ __forceinline__ float log_sigmoid_f32(float z) {
 
 template <typename T>
 __global__ void linear_prepare_kernel(const T* proj, int ld, const float* z, int ldz, const float* __restrict__ z_bias,
-                                      int kind, float p0, const int* __restrict__ token_slot, int heads, int dk, int dv,
+                                      int kind, int act, float p0, const int* __restrict__ token_slot, int heads, int dk, int dv,
                                       float q_scale, float* qn, float* kn, float* vv, float* decay, float* wgate,
                                       float* fgate) {
     TLLM_PDL_ENTER();
@@ -681,18 +689,21 @@ __global__ void linear_prepare_kernel(const T* proj, int ld, const float* z, int
     const T* row = proj + (size_t)t * ld;
     const int qk = heads * dk;
     for (int e = threadIdx.x; e < qk; e += blockDim.x) {
-        qn[(size_t)t * qk + e] = to_f32<T>(row[e]) * q_scale;
-        kn[(size_t)t * qk + e] = to_f32<T>(row[qk + e]);
+        qn[(size_t)t * qk + e] = linear_input(to_f32<T>(row[e]), act) * q_scale;
+        kn[(size_t)t * qk + e] = linear_input(to_f32<T>(row[qk + e]), act);
+    }
+    if (kind != kLinearLogGates) {
+        for (int e = threadIdx.x; e < heads * dv; e += blockDim.x)
+            vv[(size_t)t * heads * dv + e] = linear_input(to_f32<T>(row[2 * qk + e]), act);
     }
     if (kind == kLinearChannelDecay) {
-        for (int e = threadIdx.x; e < heads * dv; e += blockDim.x) vv[(size_t)t * heads * dv + e] = to_f32<T>(row[2 * qk + e]);
         for (int e = threadIdx.x; e < qk; e += blockDim.x)
             decay[(size_t)t * qk + e] = expf(p0 * log_sigmoid_f32(z[(size_t)t * ldz + e] + z_bias[e]));
-    } else {
+    } else if (kind == kLinearLogGates) {
         const int cols = dv + 1;
         for (int e = threadIdx.x; e < heads * cols; e += blockDim.x) {
             const int h = e / cols, c = e - h * cols;
-            vv[(size_t)t * heads * cols + e] = c < dv ? to_f32<T>(row[2 * qk + h * dv + c]) : 1.0f;
+            vv[(size_t)t * heads * cols + e] = c < dv ? linear_input(to_f32<T>(row[2 * qk + h * dv + c]), act) : 1.0f;
         }
         for (int h = threadIdx.x; h < heads; h += blockDim.x) {
             const float zi = z[(size_t)t * ldz + h] + z_bias[h];
@@ -700,6 +711,69 @@ __global__ void linear_prepare_kernel(const T* proj, int ld, const float* z, int
             wgate[(size_t)t * heads + h] = p0 * tanhf(zi / p0);
             fgate[(size_t)t * heads + h] = log_sigmoid_f32(p0 * tanhf(zf / p0));
         }
+    }
+}
+
+// kLinearFixedDecay with eight elements per access (every head's width a multiple of eight, everything on 16-byte
+// boundaries): a token's q | k | v is one run of pieces, dealt to gridDim.y blocks.
+template <typename T>
+__global__ void linear_prepare_vec_kernel(const T* proj, int ld, int act, const int* __restrict__ token_slot, int qk, int vd,
+                                          float q_scale, float* qn, float* kn, float* vv) {
+    TLLM_PDL_ENTER();
+    const int t = blockIdx.x;
+    if (token_slot[t] < 0) return;
+    const T* row = proj + (size_t)t * ld;
+    const int total = 2 * qk + vd;
+    for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8; c < total; c += gridDim.y * blockDim.x * 8) {
+        float v[8];
+        Ld8<T>::load(row + c, v);
+        const float scale = c < qk ? q_scale : 1.0f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = linear_input(v[e], act) * scale;
+        float* dst = c < qk ? qn + (size_t)t * qk + c : c < 2 * qk ? kn + (size_t)t * qk + (c - qk) : vv + (size_t)t * vd + (c - 2 * qk);
+        Ld8<float>::store(dst, v);
+    }
+}
+
+// ---------------------------------------------------------------- a read-out normed over all heads together
+// out = o / sqrt(mean(o^2) + eps) * weight * act(gate), the mean over a token's `width` = heads * dv numbers.  One
+// block per token; VEC: four elements per access (width and the gate's rows multiples of four, aligned).
+template <typename T, typename TG, bool VEC>
+__global__ void whole_finish_kernel(const float* o_raw, const TG* gate, int ldg, const float* __restrict__ weight, float eps,
+                                    const int* __restrict__ token_slot, int width, T* out, int gate_act) {
+    __shared__ float scratch[32];
+    TLLM_PDL_ENTER();
+    const int t = blockIdx.x;
+    T* dst = out + (size_t)t * width;
+    if (token_slot[t] < 0) {
+        for (int e = threadIdx.x; e < width; e += blockDim.x) dst[e] = from_f32<T>(0.0f);
+        return;
+    }
+    const float* src = o_raw + (size_t)t * width;
+    const TG* g = gate + (size_t)t * ldg;
+    float sum = 0.0f;
+    if (VEC) {
+        for (int e = threadIdx.x * 4; e < width; e += blockDim.x * 4) {
+            const float4 v = *reinterpret_cast<const float4*>(src + e);
+            sum += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+    } else {
+        for (int e = threadIdx.x; e < width; e += blockDim.x) sum += src[e] * src[e];
+    }
+    const float sc = 1.0f / sqrtf(block_sum(sum, scratch) / (float)width + eps);
+    if (VEC) {
+        for (int e = threadIdx.x * 4; e < width; e += blockDim.x * 4) {
+            const float4 v = *reinterpret_cast<const float4*>(src + e);
+            const float4 x = load_gate4<TG>(g + e);
+            const float4 w = *reinterpret_cast<const float4*>(weight + e);
+            dst[e] = from_f32<T>(v.x * sc * w.x * finish_gate(x.x, gate_act));
+            dst[e + 1] = from_f32<T>(v.y * sc * w.y * finish_gate(x.y, gate_act));
+            dst[e + 2] = from_f32<T>(v.z * sc * w.z * finish_gate(x.z, gate_act));
+            dst[e + 3] = from_f32<T>(v.w * sc * w.w * finish_gate(x.w, gate_act));
+        }
+    } else {
+        for (int e = threadIdx.x; e < width; e += blockDim.x)
+            dst[e] = from_f32<T>(src[e] * sc * weight[e] * finish_gate(to_f32<TG>(g[e]), gate_act));
     }
 }
 
@@ -802,22 +876,37 @@ extern "C" {
 
 // Inputs of a recurrence without a correction from the fused projections; see linear_prepare_kernel.  p0: 1 / tau
 // of the channel decays, or the cap of the gates' logits.
-int tllm_linear_prepare(const void* proj, int ld, int dtype, const float* z, int ldz, const float* z_bias, int kind,
+int tllm_linear_prepare(const void* proj, int ld, int dtype, const float* z, int ldz, const float* z_bias, int kind, int act,
                         float p0, const int* token_slot, int heads, int dk, int dv, float q_scale, float* qn, float* kn,
                         float* vv, float* decay, float* wgate, float* fgate, int n_rows, cudaStream_t stream) {
     TLLM_REQUIRE(n_rows >= 0 && heads > 0 && dk > 0 && dv > 0 && p0 > 0.0f, "linear_prepare: bad sizes");
-    TLLM_REQUIRE(kind == kLinearChannelDecay || kind == kLinearLogGates, "linear_prepare: unknown kind %d", kind);
-    TLLM_REQUIRE(ld >= 2 * heads * dk + heads * dv && ldz >= (kind == kLinearChannelDecay ? heads * dk : 2 * heads),
+    TLLM_REQUIRE(kind == kLinearChannelDecay || kind == kLinearLogGates || kind == kLinearFixedDecay, "linear_prepare: unknown kind %d", kind);
+    TLLM_REQUIRE(act == 0 || act == 1, "linear_prepare: unknown activation %d", act);
+    TLLM_REQUIRE(ld >= 2 * heads * dk + heads * dv && ldz >= (kind == kLinearChannelDecay ? heads * dk : kind == kLinearLogGates ? 2 * heads : 0),
                  "linear_prepare: rows too short");
-    TLLM_REQUIRE(kind == kLinearChannelDecay ? decay != nullptr : (wgate != nullptr && fgate != nullptr),
+    TLLM_REQUIRE(kind == kLinearChannelDecay ? decay != nullptr : kind == kLinearFixedDecay || (wgate != nullptr && fgate != nullptr),
                  "linear_prepare: no place for the gates");
     if (n_rows == 0) return 0;
+    const auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; };
+    if (kind == kLinearFixedDecay && (heads * dk) % 8 == 0 && (heads * dv) % 8 == 0 && ld % 8 == 0 && al(proj) && al(qn) && al(kn) && al(vv)) {
+        const int qk = heads * dk, vd = heads * dv, pieces = (2 * qk + vd) / 8;
+        const int sms = sm_count_cached() > 0 ? sm_count_cached() : 148;
+        int split = 1;                                  // blocks per token where few rows leave the GPU empty
+        while (split * 2 * 128 <= pieces && (long long)n_rows * split < 2LL * sms) split *= 2;
+        const dim3 grid(n_rows, split), block(128);
+        if (dtype == kBF16)
+            launch_pdl(kPdlOther, linear_prepare_vec_kernel<bf16>, grid, block, 0, stream, (const bf16*)proj, ld, act, token_slot, qk, vd, q_scale, qn, kn, vv);
+        else if (dtype == kF32)
+            launch_pdl(kPdlOther, linear_prepare_vec_kernel<float>, grid, block, 0, stream, (const float*)proj, ld, act, token_slot, qk, vd, q_scale, qn, kn, vv);
+        else TLLM_REQUIRE(false, "linear_prepare: unknown dtype %d", dtype);
+        return finish_launch("linear_prepare");
+    }
     if (dtype == kBF16)
         launch_pdl(kPdlOther, linear_prepare_kernel<bf16>, dim3(n_rows), dim3(256), 0, stream, (const bf16*)proj, ld, z, ldz,
-                   z_bias, kind, p0, token_slot, heads, dk, dv, q_scale, qn, kn, vv, decay, wgate, fgate);
+                   z_bias, kind, act, p0, token_slot, heads, dk, dv, q_scale, qn, kn, vv, decay, wgate, fgate);
     else if (dtype == kF32)
         launch_pdl(kPdlOther, linear_prepare_kernel<float>, dim3(n_rows), dim3(256), 0, stream, (const float*)proj, ld, z, ldz,
-                   z_bias, kind, p0, token_slot, heads, dk, dv, q_scale, qn, kn, vv, decay, wgate, fgate);
+                   z_bias, kind, act, p0, token_slot, heads, dk, dv, q_scale, qn, kn, vv, decay, wgate, fgate);
     else TLLM_REQUIRE(false, "linear_prepare: unknown dtype %d", dtype);
     return finish_launch("linear_prepare");
 }
@@ -946,10 +1035,11 @@ int tllm_delta_scan(const int* seg_info, int segments, int rows, const int* toke
                     const float* erase, long long aux_off, float floor_eps, float* den, cudaStream_t stream) {
     TLLM_REQUIRE(segments >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dk > 0 && dv > 0,
                  "delta_scan: bad sizes");
-    TLLM_REQUIRE(mode == kScanDelta || mode == kScanPlain || mode == kScanMemory || mode == kScanHeadDecay || mode == kScanErase,
+    TLLM_REQUIRE(mode == kScanDelta || mode == kScanPlain || mode == kScanMemory || mode == kScanHeadDecay || mode == kScanErase ||
+                 mode == kScanFixedDecay,
                  "delta_scan: unknown recurrence %d", mode);
     TLLM_REQUIRE(mode == kScanMemory ? (beta != nullptr && fgate != nullptr && den != nullptr && dv >= 2 && aux_off > 0)
-                 : mode == kScanHeadDecay ? (beta != nullptr && fgate != nullptr) : decay != nullptr, "delta_scan: the recurrence lacks an operand");
+                 : mode == kScanHeadDecay ? (beta != nullptr && fgate != nullptr) : mode == kScanFixedDecay ? fgate != nullptr : decay != nullptr, "delta_scan: the recurrence lacks an operand");
     TLLM_REQUIRE(mode != kScanDelta || beta != nullptr, "delta_scan: the delta rule needs its betas");
     TLLM_REQUIRE(mode != kScanErase || (erase != nullptr && kv_heads == heads), "delta_scan: a removal per channel needs its rates and a key per head");
     TLLM_REQUIRE(heads <= 65535, "delta_scan: %d heads", heads);
@@ -980,6 +1070,7 @@ int tllm_delta_scan(const int* seg_info, int segments, int rows, const int* toke
         else if (mode == kScanPlain) SCAN_MODE(RR, PP, kScanPlain);                                              \
         else if (mode == kScanHeadDecay) SCAN_MODE(RR, PP, kScanHeadDecay);                                      \
         else if (mode == kScanErase) SCAN_MODE(RR, PP, kScanErase);                                              \
+        else if (mode == kScanFixedDecay) SCAN_MODE(RR, PP, kScanFixedDecay);                                    \
         else SCAN_MODE(RR, PP, kScanMemory);                                                                     \
     } while (0)
 #define SCAN_MODE(RR, PP, MM)                                                                                           \
@@ -1011,6 +1102,30 @@ int tllm_delta_scan(const int* seg_info, int segments, int rows, const int* toke
 #undef SCAN_MODE
 #undef SCAN_NC
     return finish_launch("delta_scan");
+}
+
+// The read-out of all heads normed together; see whole_finish_kernel.  gate: float32 (gate_f32) or the storage type.
+int tllm_whole_finish(const float* o_raw, const void* gate, int gate_f32, int ldg, const float* weight, float eps,
+                      const int* token_slot, int n_rows, int width, void* out, int dtype, int gate_act, cudaStream_t stream) {
+    TLLM_REQUIRE(n_rows >= 0 && width > 0 && eps > 0.0f && ldg >= width, "whole_finish: bad sizes");
+    TLLM_REQUIRE(gate_act == 0 || gate_act == 1, "whole_finish: bad options");
+    if (n_rows == 0) return 0;
+    const auto al = [](const void* p, unsigned to) { return (reinterpret_cast<uintptr_t>(p) & (to - 1)) == 0; };
+    const bool vec = width % 4 == 0 && ldg % 4 == 0 && al(o_raw, 16) && al(weight, 16) && al(gate, gate_f32 || dtype == kF32 ? 16 : 8);
+    int threads = 64;                                   // about two accesses of four per thread
+    while (threads < 512 && threads * 8 < width) threads *= 2;
+#define WHOLE(T, TG)                                                                                                        \
+    do {                                                                                                                    \
+        if (vec) launch_pdl(kPdlOther, whole_finish_kernel<T, TG, true>, dim3(n_rows), dim3(threads), 0, stream, o_raw,      \
+                            (const TG*)gate, ldg, weight, eps, token_slot, width, (T*)out, gate_act);                       \
+        else launch_pdl(kPdlOther, whole_finish_kernel<T, TG, false>, dim3(n_rows), dim3(threads), 0, stream, o_raw,         \
+                        (const TG*)gate, ldg, weight, eps, token_slot, width, (T*)out, gate_act);                           \
+    } while (0)
+    if (dtype == kBF16) { if (gate_f32) WHOLE(bf16, float); else WHOLE(bf16, bf16); }
+    else if (dtype == kF32) WHOLE(float, float);
+    else TLLM_REQUIRE(false, "whole_finish: unknown dtype %d", dtype);
+#undef WHOLE
+    return finish_launch("whole_finish");
 }
 
 // gate: float32 (gate_f32) or the storage type; state_dv: value columns of S in the state's layout (dv, or more where

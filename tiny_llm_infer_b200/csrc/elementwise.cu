@@ -1131,7 +1131,7 @@ int tllm_postnorm_add_rmsnorm(float* h, const void* delta, const void* post_gain
 int tllm_swiglu(const void* gate_up, void* out, int dtype, int tokens, int inter, int interleaved,
                 int act, float limit, float slope, cudaStream_t stream) {
     const GateConst gc{limit, slope};
-    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh || (act == kActClampedSwish && limit > 0.0f), "swiglu: unknown activation %d", act);
+    TLLM_REQUIRE(gated_act_ok(act, limit), "swiglu: unknown activation %d", act);
     TLLM_REQUIRE(tokens >= 0 && inter > 0, "swiglu: bad sizes");
     TLLM_REQUIRE(!interleaved || inter % 8 == 0, "swiglu: interleaved columns need a multiple of 8, not %d", inter);
     TLLM_REQUIRE(dtype == kBF16 || dtype == kF32, "swiglu: unknown dtype %d", dtype);

@@ -231,11 +231,11 @@ extern "C" int tllm_gemm_skinny(const void* x, const void* w, void* y, int out_d
     return launch_skinny<4, float, false>(x, w, y, M, N, K, stream);
 }
 
-// y[M, N] = act(x . gate^T) * (x . up^T), act silu, the tanh form of GELU or the clamped swish (with its constants),
+// y[M, N] = act(x . gate^T) * (x . up^T), act silu, the tanh form of GELU, ReLU or the clamped swish (with its constants),
 // for w of 2 N rows, gate and up interleaved by eight (eight gate rows, their eight up rows, ...), bfloat16 out, M <= 16.
 extern "C" int tllm_gemm_skinny_swiglu(const void* x, const void* w, void* y, int M, int N, int K, int act,
                                        float limit, float slope, cudaStream_t stream) {
-    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh || (act == kActClampedSwish && limit > 0.0f), "gemm_skinny_swiglu: unknown activation %d", act);
+    TLLM_REQUIRE(gated_act_ok(act, limit), "gemm_skinny_swiglu: unknown activation %d", act);
     TLLM_REQUIRE(M >= 0 && N > 0 && K > 0, "gemm_skinny_swiglu: bad sizes");
     TLLM_REQUIRE(M <= 16, "gemm_skinny_swiglu: %d rows exceed 16", M);
     TLLM_REQUIRE(N % 8 == 0, "gemm_skinny_swiglu: N = %d is no multiple of 8", N);
@@ -246,6 +246,10 @@ extern "C" int tllm_gemm_skinny_swiglu(const void* x, const void* w, void* y, in
     if (act == kActGeluTanh) {
         if (M <= 8) return launch_skinny<1, bf16, true, 3, kActGeluTanh>(x, w, y, M, N, K, stream);
         return launch_skinny<2, bf16, true, 3, kActGeluTanh>(x, w, y, M, N, K, stream);
+    }
+    if (act == kActRelu) {
+        if (M <= 8) return launch_skinny<1, bf16, true, 3, kActRelu>(x, w, y, M, N, K, stream);
+        return launch_skinny<2, bf16, true, 3, kActRelu>(x, w, y, M, N, K, stream);
     }
     if (act == kActClampedSwish) {
         const GateConst gc{limit, slope};

@@ -38,10 +38,11 @@ constexpr int kGemmThreads = 192;
 constexpr uint32_t kTmemCols = 512;
 constexpr int kSpinLimit = 1 << 20;
 
-// act(gate) of the gated epilogue with the fast intrinsics: silu g / (1 + e^-g), or the tanh form of GELU
-// written the same way, 0.5 g (1 + tanh(u)) = g / (1 + e^-2u) with u = sqrt(2/pi) (g + 0.044715 g^3).
+// act(gate) of the gated epilogue with the fast intrinsics: silu g / (1 + e^-g), the tanh form of GELU
+// written the same way, 0.5 g (1 + tanh(u)) = g / (1 + e^-2u) with u = sqrt(2/pi) (g + 0.044715 g^3), or ReLU.
 template <int ACT>
 __device__ __forceinline__ float fast_gate_act(float g) {
+    if (ACT == kActRelu) return fmaxf(g, 0.0f);
     if (ACT == kActGeluTanh) {
         const float u2 = 1.5957691216057308f * (g + 0.044715f * g * g * g);
         return __fdividef(g, 1.0f + __expf(-u2));
@@ -530,13 +531,16 @@ extern "C" int tllm_gemm_tcgen05(const void* x, const void* w, void* y, int M, i
 #undef UNARY
         TLLM_REQUIRE(false, "gemm_tcgen05: unknown activation %d", act);
     }
-    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh || (act == kActClampedSwish && limit > 0.0f), "gemm_tcgen05: unknown activation %d", act);
+    TLLM_REQUIRE(gated_act_ok(act, limit), "gemm_tcgen05: unknown activation %d", act);
     if ((swiglu & 1) && act == kActClampedSwish) {
         const GateConst gc{limit, slope};
         const GroupedTiles plain{nullptr, nullptr, nullptr, nullptr, 0};
         return tall ? launch_tcgen05<true, 2, kActClampedSwish>(mx, mw, y, M, N, K, N / 2, interleaved, error_word, stream, plain, 0, gc)
                     : launch_tcgen05<true, 1, kActClampedSwish>(mx, mw, y, M, N, K, N / 2, interleaved, error_word, stream, plain, 0, gc);
     }
+    if ((swiglu & 1) && act == kActRelu)
+        return tall ? launch_tcgen05<true, 2, kActRelu>(mx, mw, y, M, N, K, N / 2, interleaved, error_word, stream)
+                    : launch_tcgen05<true, 1, kActRelu>(mx, mw, y, M, N, K, N / 2, interleaved, error_word, stream);
     if ((swiglu & 1) && act == kActGeluTanh)
         return tall ? launch_tcgen05<true, 2, kActGeluTanh>(mx, mw, y, M, N, K, N / 2, interleaved, error_word, stream)
                     : launch_tcgen05<true, 1, kActGeluTanh>(mx, mw, y, M, N, K, N / 2, interleaved, error_word, stream);
@@ -578,10 +582,12 @@ extern "C" int tllm_gemm_tcgen05_grouped(const void* x, const void* w, void* y, 
 #undef UNARY
         TLLM_REQUIRE(false, "gemm_tcgen05_grouped: unknown activation %d", act);
     }
-    TLLM_REQUIRE(act == kActSilu || act == kActGeluTanh || (act == kActClampedSwish && limit > 0.0f), "gemm_tcgen05_grouped: unknown activation %d", act);
+    TLLM_REQUIRE(gated_act_ok(act, limit), "gemm_tcgen05_grouped: unknown activation %d", act);
     if (gated && act == kActClampedSwish)
         return launch_tcgen05<true, 1, kActClampedSwish>(mx, mw, y, rows, n, K, n / 2, 1, error_word, stream, grouped, max_tiles,
                                                          GateConst{limit, slope});
+    if (gated && act == kActRelu)
+        return launch_tcgen05<true, 1, kActRelu>(mx, mw, y, rows, n, K, n / 2, 1, error_word, stream, grouped, max_tiles);
     if (gated && act == kActGeluTanh)
         return launch_tcgen05<true, 1, kActGeluTanh>(mx, mw, y, rows, n, K, n / 2, 1, error_word, stream, grouped, max_tiles);
     if (gated) return launch_tcgen05<true, 1>(mx, mw, y, rows, n, K, n / 2, 1, error_word, stream, grouped, max_tiles);

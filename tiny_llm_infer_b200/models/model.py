@@ -103,12 +103,13 @@ class Model:
     def workspace_floats(self, tokens: int, wanted: int) -> int:
         """Float32 words (an upper estimate) of the activations alive at once in a step of ``tokens``
         rows of which ``wanted`` get logits: the residual stream and a handful of rows of the model's
-        width, plus the widest thing any one part makes.  A part says what it makes with
+        width, plus the widest thing any one part makes and what parts leave for later ones (``kept_floats(tokens)``).  A part says what it makes with
         ``workspace_floats(tokens)``; one that does not is taken to stay within the model's width."""
         widest = max([0] + [int(part.workspace_floats(tokens)) for part in self.parts()
                             if part is not self.head and hasattr(part, "workspace_floats")])
         head = int(self.head.workspace_floats(wanted)) if hasattr(self.head, "workspace_floats") else wanted * self.desc.vocab_size
-        return 6 * tokens * self.desc.hidden_size + widest + head
+        kept = sum(int(part.kept_floats(tokens)) for part in self.parts() if hasattr(part, "kept_floats"))
+        return 6 * tokens * self.desc.hidden_size + widest + head + kept
 
     # ---- one step
     def forward(self, ctx, caches) -> torch.Tensor:

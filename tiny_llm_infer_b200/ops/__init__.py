@@ -64,7 +64,7 @@ def _declare(h) -> None:
         "tllm_embedding": [vp, vp, i32, vp, i32, i32, i32, f32, vp],
         "tllm_postnorm_add_rmsnorm": [vp, vp, vp, f32, vp, i32, f32, vp, i32, vp, i32, i32, vp],
         "tllm_qkv_unit_store": [vp, i32, vp, vp, f32, i32, vp, vp, vp, i32, i32, vp, vp, i64, vp, i32, i32,
-                                i32, i32, i32, i32, i32, vp, i32, f32, i32, i32, vp, vp],
+                                i32, i32, i32, i32, i32, vp, i32, i32, f32, i32, i32, vp, vp, i32, vp, f32, vp],
         "tllm_attention_biased_general": [vp, vp, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32,
                                           f32, f32, i32, i32, i32, vp, vp, vp, i32, i32, vp, i32, i32, i32, f32, f32, f32, vp, vp],
         "tllm_attention_biased_prefill": [vp, vp, vp, i64, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32,
@@ -72,7 +72,8 @@ def _declare(h) -> None:
         "tllm_attention_biased_decode": [vp, vp, vp, i64, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, i32,
                                          f32, f32, i32, i32, i32, vp, vp, vp, i32, i32, vp, i32, i32, i32, f32, f32, f32, i32, vp, vp, vp],
         "tllm_scaled_add_layernorm": [vp, vp, vp, i32, vp, i32, f32, vp, i32, vp, i32, i32, vp],
-        "tllm_linear_prepare": [vp, i32, i32, vp, i32, vp, i32, f32, vp, i32, i32, i32, f32, vp, vp, vp, vp, vp, vp,
+        "tllm_whole_finish": [vp, vp, i32, i32, vp, f32, vp, i32, i32, vp, i32, i32, vp],
+        "tllm_linear_prepare": [vp, i32, i32, vp, i32, vp, i32, i32, f32, vp, i32, i32, i32, f32, vp, vp, vp, vp, vp, vp,
                                 i32, vp],
         "tllm_embedding_norm": [vp, vp, vp, vp, i32, vp, f32, f32, vp, i32, i32, i32, i32, vp],
         "tllm_softcap": [vp, f32, i64, vp],
@@ -271,7 +272,7 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
     return torch.stack([gate.reshape(inter // 8, 8, k), up.reshape(inter // 8, 8, k)], dim=1).reshape(2 * inter, k)
 
 
-ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 4}      # of gated units: codes of csrc/common.cuh (GateAct)
+ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 4, "relu": 6}      # of gated units: codes of csrc/common.cuh (GateAct)
 NO_CONSTS = (0.0, 0.0)       # ``consts``: (limit, slope) of ``clamped_swish``, g sigmoid(slope g) (u + 1) with g = min(gate,
                              # limit) and u = up held within -limit .. limit; the other activations have none
 
@@ -287,7 +288,7 @@ def swiglu(gate_up: torch.Tensor, out: torch.Tensor, interleaved: bool = False, 
            consts=None) -> torch.Tensor:
     """out[t, i] = act(gate) * up with gate = gate_up[t, i], up = gate_up[t, I + i], or, for columns
     interleaved by eight, gate = gate_up[t, 16 (i // 8) + i % 8] and up eight columns further.
-    ``act``: ``silu``, ``gelu_tanh`` or ``clamped_swish`` (with its ``consts``)."""
+    ``act``: ``silu``, ``gelu_tanh``, ``relu`` or ``clamped_swish`` (with its ``consts``)."""
     _cuda(gate_up, out)
     tokens, two_i = gate_up.shape
     assert out.shape == (tokens, two_i // 2) and out.dtype == gate_up.dtype
@@ -700,12 +701,16 @@ def biased_decode_splits(rows: int, kv_heads: int, reach: int) -> int:
     return max(1, min(want, reach // 256, 64))
 
 
+QK_WHOLE = 2             # norm of all heads together (csrc/attention_biased.cu, QkNorm)
+
+
 def qkv_unit_store(proj: torch.Tensor, q_out: torch.Tensor, positions, token_slot, block_table,
                    k_plane: Optional[torch.Tensor], v_plane: Optional[torch.Tensor], page_size: int,
                    q_heads: int, kv_heads: int, dk: int, dv: int, eps: Optional[float],
                    q_gain: Optional[torch.Tensor] = None, k_gain: Optional[torch.Tensor] = None,
                    store: bool = True, inv_freq: Optional[torch.Tensor] = None, rot_dims: int = 0,
-                   q_temperature=None, values_are_keys: bool = False, bias: Optional[torch.Tensor] = None) -> None:
+                   q_temperature=None, values_are_keys: bool = False, bias: Optional[torch.Tensor] = None,
+                   norm_whole: bool = False, rot_pairs: bool = False, value_mix=None) -> None:
     """Rows of ``proj`` = q heads | k heads | v heads | anything: queries and keys divided per head by
     their root mean square (``eps`` None: left as they are; gains optional), queries to ``q_out``,
     keys and values of every row into their planes of the paged cache (``store``).  Keys have width
@@ -713,7 +718,11 @@ def qkv_unit_store(proj: torch.Tensor, q_out: torch.Tensor, positions, token_slo
     ``rot_dims`` elements of every query and key head turn by position * inv_freq (pairs half the rotated width
     apart), after the norm.  ``q_temperature`` (coef, every): queries times 1 + coef ln(floor((pos + 1) / every) + 1).
     ``values_are_keys``: the rows carry no values; a value is its key as projected, before the norm (dv = dk).
-    ``bias`` float32, one number per q | k | v column: added to the rows, in float32, before anything else."""
+    ``bias`` float32, one number per q | k | v column: added to the rows, in float32, before anything else.
+    ``norm_whole``: the queries of a row are normed as one vector of all heads, and so are its keys; the gains then
+    have q_heads * dk and kv_heads * dk numbers.  ``rot_pairs``: elements 2 i and 2 i + 1 turn together.
+    ``value_mix`` (other, its bias or None, share): values become (1 - share) v + share (other + bias) before they
+    are written, with ``other`` [T, kv_heads * dv] the values of the same rows elsewhere (a view, rows may be strided)."""
     _cuda(proj, q_out, positions, token_slot, block_table, q_gain, k_gain, inv_freq, bias)
     if bias is not None:
         assert bias.dtype == torch.float32 and bias.numel() == (q_heads + kv_heads) * dk + (0 if values_are_keys else kv_heads * dv)
@@ -721,6 +730,13 @@ def qkv_unit_store(proj: torch.Tensor, q_out: torch.Tensor, positions, token_slo
         assert inv_freq.dtype == torch.float32 and inv_freq.numel() == rot_dims // 2
     if q_gain is not None:
         assert q_gain.dtype == k_gain.dtype == proj.dtype
+        assert (q_gain.numel(), k_gain.numel()) == ((q_heads * dk, kv_heads * dk) if norm_whole else (dk, dk))
+    other, other_bias, share = value_mix if value_mix is not None else (None, None, 0.0)
+    if other is not None:
+        assert other.is_cuda and other.dtype == proj.dtype and other.stride(1) == 1
+        assert tuple(other.shape) == (proj.shape[0], kv_heads * dv)
+        if other_bias is not None:
+            assert other_bias.dtype == torch.float32 and other_bias.is_contiguous() and other_bias.numel() == kv_heads * dv
     coef, every = q_temperature if q_temperature is not None else (0.0, 0)
     assert q_out.dtype == proj.dtype and tuple(q_out.shape) == (proj.shape[0], q_heads * dk)
     kp = vp = None
@@ -731,11 +747,13 @@ def qkv_unit_store(proj: torch.Tensor, q_out: torch.Tensor, positions, token_slo
         (kp, stride), (vp, stride_v) = _plane(k_plane), _plane(v_plane)
         assert stride == stride_v
     _check(lib().tllm_qkv_unit_store(
-        _p(proj), proj.shape[1], _p(q_gain), _p(k_gain), float(eps or 1.0), int(eps is not None), _p(positions),
+        _p(proj), proj.shape[1], _p(q_gain), _p(k_gain), float(eps or 1.0),
+        QK_WHOLE if eps is not None and norm_whole else int(eps is not None), _p(positions),
         _p(token_slot), _p(block_table), block_table.shape[1] if block_table is not None else 0, page_size,
         kp, vp, stride, _p(q_out), _dt(proj), proj.shape[0], q_heads, kv_heads, dk, dv, int(store),
-        _p(inv_freq), int(rot_dims if inv_freq is not None else 0), float(coef), int(every), int(values_are_keys),
-        _p(bias), _stream()), "qkv_unit_store")
+        _p(inv_freq), int(rot_dims if inv_freq is not None else 0), int(rot_pairs), float(coef), int(every),
+        int(values_are_keys), _p(bias), None if other is None else other.data_ptr(),
+        0 if other is None else other.stride(0), _p(other_bias), float(share), _stream()), "qkv_unit_store")
 
 
 def attention_biased(q: torch.Tensor, k_plane: torch.Tensor, v_plane: torch.Tensor, positions, token_slot,
@@ -978,7 +996,8 @@ def delta_rule_state_floats(heads: int, kv_heads: int, dk: int, dv: int, taps: i
     return int(lib().tllm_delta_rule_state_floats(heads, kv_heads, dk, dv, taps))
 
 
-SCAN_DELTA, SCAN_PLAIN, SCAN_MEMORY, SCAN_HEAD_DECAY, SCAN_ERASE = 0, 1, 2, 3, 4     # recurrences of the scan kernel (csrc/delta_rule.cu, ScanMode)
+SCAN_DELTA, SCAN_PLAIN, SCAN_MEMORY, SCAN_HEAD_DECAY, SCAN_ERASE, SCAN_FIXED_DECAY = 0, 1, 2, 3, 4, 5     # recurrences of the scan kernel (csrc/delta_rule.cu, ScanMode)
+INPUT_ACTS = {None: 0, "silu": 1}                     # of q, k and v before a recurrence without a correction
 GATE_ACTS = {"sigmoid": 0, "silu": 1}                # what the read-out is multiplied by: act(gate)
 
 
@@ -1075,7 +1094,7 @@ def erase_delta_rule(proj: torch.Tensor, a_col: int, z: torch.Tensor, z_bias: to
                          out_dtype, None, 0, 1, state, None, gate_act)
 
 
-LINEAR_KINDS = {"channel_decay": 0, "log_gates": 1}      # csrc/delta_rule.cu, LinearKind
+LINEAR_KINDS = {"channel_decay": 0, "log_gates": 1, "fixed_decay": 2}      # csrc/delta_rule.cu, LinearKind
 
 
 def linear_recurrence_state_floats(kind: str, heads: int, dk: int, dv: int) -> int:
@@ -1086,10 +1105,11 @@ def linear_recurrence_state_floats(kind: str, heads: int, dk: int, dv: int) -> i
     return s_floats + (heads * cols if kind == "log_gates" else 0)
 
 
-def linear_recurrence(proj: torch.Tensor, kind: str, z: torch.Tensor, z_bias: torch.Tensor, p0: float,
+def linear_recurrence(proj: torch.Tensor, kind: str, z: Optional[torch.Tensor], z_bias: torch.Tensor, p0: float,
                       gate: torch.Tensor, gate_act: str, out_weight: torch.Tensor, weight_per_head: bool, eps: float,
                       token_slot: torch.Tensor, seg_info: Optional[torch.Tensor], state: torch.Tensor, heads: int,
-                      dk: int, dv: int, q_scale: float, out_dtype: torch.dtype, floor_eps: float = 1e-6) -> torch.Tensor:
+                      dk: int, dv: int, q_scale: float, out_dtype: torch.dtype, floor_eps: float = 1e-6,
+                      input_act: Optional[str] = None, norm_whole: bool = False) -> torch.Tensor:
     """One step of a recurrence S <- decay S + k (w v)^T, o = S^T q per head, for every row of ``proj`` [T, >= heads
     (2 dk + dv)] = q | k | v in the storage type (q is multiplied by ``q_scale``), from ``state[slot]`` (float32,
     updated in place).  ``kind``:
@@ -1098,15 +1118,20 @@ def linear_recurrence(proj: torch.Tensor, kind: str, z: torch.Tensor, z_bias: to
     * ``log_gates``: ``z`` [T, 2 heads] float32 = write | keep logits (plus ``z_bias``), each capped as p0 tanh(. /
       p0); with i the capped write logit and f = logsigmoid(capped keep logit), a running maximum m <- max(f + m, i)
       that starts at zero: decay = exp(f + m_before - m), w = exp(i - m); a vector n <- decay n + w k is kept beside
-      S and the read-out is S^T q / (max(|n . q|, exp(-m)) + ``floor_eps``).
+      S and the read-out is S^T q / (max(|n . q|, exp(-m)) + ``floor_eps``);
+    * ``fixed_decay``: no ``z``; ``z_bias`` [heads] float32 holds every head's decay itself, w = 1.
 
-    Then the read-out is divided by its root mean square per head (``eps``), times ``out_weight`` ([dv], or [heads *
+    ``input_act`` ``silu``: q (before its scale), k and v are SiLU of what is in ``proj``.  Then the read-out is divided by its root mean square per head (``eps``), times ``out_weight`` ([dv], or [heads *
     dv] with ``weight_per_head``) float32, times ``gate_act``(``gate``) ([T, heads * dv], rows may be strided).
-    Returns [T, heads * dv] in ``out_dtype``."""
+    ``norm_whole``: the root mean square is the one of all heads together (``weight_per_head``, no divisor).  Returns [T, heads * dv] in ``out_dtype``."""
     _cuda(proj, z_bias, out_weight, token_slot, seg_info, state)
     tokens, ld = proj.shape
-    assert z.dtype == z_bias.dtype == state.dtype == torch.float32 and z.stride(1) == 1 and state.dim() == 2
-    memory = kind == "log_gates"
+    assert z_bias.dtype == state.dtype == torch.float32 and state.dim() == 2
+    memory, fixed = kind == "log_gates", kind == "fixed_decay"
+    if fixed:
+        assert z is None and z_bias.numel() == heads
+    else:
+        assert z.dtype == torch.float32 and z.stride(1) == 1
     cols = dv + 1 if memory else dv
     assert state.shape[1] == linear_recurrence_state_floats(kind, heads, dk, dv)
     dev = proj.device
@@ -1119,18 +1144,27 @@ def linear_recurrence(proj: torch.Tensor, kind: str, z: torch.Tensor, z_bias: to
         at += -(-tokens * n // 4) * 4
         return t
     qn, kn = take(heads * dk), take(heads * dk)
-    decay = None if memory else take(heads * dk)
+    decay = None if memory or fixed else take(heads * dk)
     vv, o_raw = take(heads * cols), take(heads * dv)
     wgate, fgate, den = (take(heads), take(heads), take(heads)) if memory else (None, None, None)
-    _check(lib().tllm_linear_prepare(_p(proj), ld, _dt(proj), z.data_ptr(), z.stride(0), _p(z_bias), LINEAR_KINDS[kind],
-                                     float(p0), _p(token_slot), heads, dk, dv, float(q_scale), _p(qn), _p(kn), _p(vv),
+    _check(lib().tllm_linear_prepare(_p(proj), ld, _dt(proj), None if fixed else z.data_ptr(), 0 if fixed else z.stride(0), _p(z_bias),
+                                     LINEAR_KINDS[kind], INPUT_ACTS[input_act], float(p0), _p(token_slot), heads, dk, dv, float(q_scale), _p(qn), _p(kn), _p(vv),
                                      _p(decay), _p(wgate), _p(fgate), tokens, _stream()), "linear_prepare")
     segments = tokens if seg_info is None else seg_info.shape[0]
     aux_off = delta_rule_state_floats(heads, heads, dk, cols, 1) if memory else 0
     _check(lib().tllm_delta_scan(_p(seg_info), segments, tokens, _p(token_slot), _p(qn), _p(kn), _p(vv), _p(decay), _p(wgate),
                                  _p(state), state.stride(0), heads, heads, dk, cols, _p(o_raw),
-                                 SCAN_MEMORY if memory else SCAN_PLAIN, _p(fgate), None, aux_off, float(floor_eps), _p(den),
-                                 _stream()), "delta_scan")
+                                 SCAN_MEMORY if memory else SCAN_FIXED_DECAY if fixed else SCAN_PLAIN,
+                                 _p(z_bias) if fixed else _p(fgate), None, aux_off, float(floor_eps), _p(den), _stream()),
+           "delta_scan")
+    if norm_whole:
+        assert weight_per_head and den is None and gate.stride(1) == 1 and gate.dtype in (torch.float32, out_dtype)
+        assert out_weight.dtype == torch.float32 and out_weight.numel() == heads * dv == gate.shape[1]
+        out = torch.empty((tokens, heads * dv), dtype=out_dtype, device=dev)
+        _check(lib().tllm_whole_finish(_p(o_raw), gate.data_ptr(), int(gate.dtype == torch.float32), gate.stride(0), _p(out_weight),
+                                       float(eps), _p(token_slot), tokens, heads * dv, _p(out), _dt(out), GATE_ACTS[gate_act],
+                                       _stream()), "whole_finish")
+        return out
     return _delta_finish(o_raw, gate, out_weight, weight_per_head, eps, token_slot, tokens, heads, heads, dk, dv,
                          out_dtype, None, 0, 1, state, den, gate_act)
 

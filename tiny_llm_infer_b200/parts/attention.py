@@ -43,6 +43,8 @@ class GroupedQueryAttention:
         self.position = None
         if position is not None:
             self.position = lookup("position", position.kind)(dtype=dtype, device=device, **position.params)
+            if getattr(self.position, "pairs", False):
+                raise ValueError(f"position encoding {position.kind!r} turns neighbouring elements, this part's kernel halves")
         self.w_qkv = self.w_o = self.q_gain = self.k_gain = None
 
     # ---- weights

@@ -3,9 +3,14 @@ softmax, with an output gate.  Every step is a parameter, so other designs can p
 
   q, k        per head divided by their root mean square over the head (``unit_norm_eps``; None: not), then,
               with ``qk_gains``, multiplied by a learned gain of the head's width (tensors ``<q>.norm``, ``<k>.norm``,
-              shared by the heads); ``position`` (a part of the position registry that the norm kernel can apply
-              itself, such as ``rotary_half`` over part of the head): q and k turned by their positions
-  values      projected by Wv, or, ``values_are_keys``, the keys as projected, before their norm (no Wv)
+              shared by the heads); with ``norm_whole`` the root mean square is the one of all heads together, of
+              the queries and of the keys, and the gains have a number per row of the projection; ``position`` (a
+              part of the position registry that the norm kernel can apply itself, such as ``rotary_half`` or
+              ``rotary_pairs`` over part of the head): q and k turned by their positions
+  values      projected by Wv, or, ``values_are_keys``, the keys as projected, before their norm (no Wv);
+              ``value_mix``: a model's first layer that says so leaves its values (``"first"``) and every later one
+              takes them in (``"mix"``), v <- (1 - c) v + c v_first with a learned number c (tensor
+              ``value_mix_name``, which the first layer has too and does not use); the mixed values are what is cached
   temperature ``q_temperature`` (coef, every): the query at position p times 1 + coef ln(floor((p + 1) / every) + 1)
   score       s = (q . k) * scale;  ``softcap`` c: s <- c tanh(s / c);  ``bias_slopes`` m_h: s <- s - m_h (i - j)
               (``slope_exponent`` e instead of explicit slopes: m_h = 2^(-e (h + 1) / heads));
@@ -24,7 +29,8 @@ softmax, with an output gate.  Every step is a parameter, so other designs can p
               ``difference_names``) the head is o = a1 - lambda a2, then o / sqrt(mean(o^2) + eps) (1 - diff)
   biases      ``biases``: q, k, v and the output product have biases (tensors ``<name>`` + ``bias_suffix``), added in
               float32 where the norm kernel reads the projections; the output's is added by the product, or, with
-              ``defer_output_bias``, left as ``deferred_bias`` for the block's sum kernel to add
+              ``defer_output_bias``, left as ``deferred_bias`` for the block's sum kernel to add; without
+              ``output_bias`` the output product has none
 
 Keys have width ``key_dim`` and values ``value_dim``; they are two planes of the paged cache.  With a
 chunk or a window the cache keeps only the keys a later query can still see (a chunk never reaches
@@ -69,6 +75,7 @@ class BiasedAttention:
     graph_safe = True
     NAMES = ("q", "k", "v", "o", "g")
     DIFFERENCE_NAMES = ("lq1", "lk1", "lq2", "lk2")
+    FIRST_VALUES = "first_values"      # key of the step's memo: the values that later layers mix into theirs
 
     def __init__(self, hidden_size: int, q_heads: int, kv_heads: int, key_dim: int, value_dim: int,
                  scale: float, dtype: torch.dtype, device, unit_norm_eps: Optional[float] = None,
@@ -81,7 +88,9 @@ class BiasedAttention:
                  distance_bias: Optional[Tuple[int, float]] = None, bias_name: str = "rel",
                  learned_sink: bool = False, sink_name: str = "sink", gate_per_head: bool = False,
                  biases: bool = False, bias_suffix: str = ".b", defer_output_bias: bool = False,
-                 differential: Optional[Tuple[float, float]] = None, difference_names: Sequence[str] = DIFFERENCE_NAMES):
+                 differential: Optional[Tuple[float, float]] = None, difference_names: Sequence[str] = DIFFERENCE_NAMES,
+                 output_bias: bool = True, norm_whole: bool = False, value_mix: Optional[str] = None,
+                 value_mix_name: str = "vmix"):
         if q_heads % kv_heads:
             raise ValueError(f"{q_heads} query heads cannot share {kv_heads} key/value heads")
         if unit_norm_eps is not None and not unit_norm_eps > 0.0:
@@ -107,6 +116,14 @@ class BiasedAttention:
         self.qk_gains, self.gain_suffix = bool(qk_gains), gain_suffix
         if self.qk_gains and unit_norm_eps is None:
             raise ValueError("gains on queries and keys come with their norm: give unit_norm_eps")
+        self.norm_whole = bool(norm_whole)
+        if self.norm_whole and unit_norm_eps is None:
+            raise ValueError("a norm over all heads is a norm: give unit_norm_eps")
+        if value_mix not in (None, "first", "mix"):
+            raise ValueError(f"value_mix is 'first', 'mix' or None, got {value_mix!r}")
+        self.value_mix, self.value_mix_name, self.value_share = value_mix, value_mix_name, 0.0
+        if value_mix is not None and values_are_keys:
+            raise ValueError("values that are keys are not mixed with another layer's")
         self.values_are_keys = bool(values_are_keys)
         if self.values_are_keys and key_dim != value_dim:
             raise ValueError(f"keys of width {key_dim} cannot be values of width {value_dim}")
@@ -124,16 +141,18 @@ class BiasedAttention:
         self.learned_sink, self.sink_name = bool(learned_sink), sink_name
         if self.learned_sink and not self.sink:
             raise ValueError("a learned sink is a sink: give sink=True")
-        self.inv_freq, self.rot_dims = None, 0
+        self.inv_freq, self.rot_dims, self.rot_pairs = None, 0, False
         if position is not None:
             part = lookup("position", position.kind)(dtype=dtype, device=device, **position.params)
             if not hasattr(part, "fused_rotary"):
                 raise ValueError(f"position encoding {position.kind!r} cannot be applied by the norm kernel")
             self.inv_freq, self.rot_dims = part.fused_rotary()
+            self.rot_pairs = bool(getattr(part, "pairs", False))
             if self.rot_dims > key_dim:
                 raise ValueError(f"a rotation of {self.rot_dims} elements in heads of {key_dim}")
         self.gate_per_head, self.biases, self.bias_suffix = bool(gate_per_head), bool(biases), bias_suffix
-        self.defer_output_bias = bool(defer_output_bias) and self.biases
+        self.output_bias = bool(output_bias) and self.biases
+        self.defer_output_bias = bool(defer_output_bias) and self.output_bias
         if self.gate_per_head and not self.output_gate:
             raise ValueError("a gate per head is an output gate: give output_gate=True")
         self.maps, self.differential, self.difference_names = 1, None, tuple(difference_names)
@@ -153,7 +172,8 @@ class BiasedAttention:
     def param_specs(cls, hidden_size, q_heads, kv_heads, key_dim, value_dim, output_gate=False,
                     names=NAMES, qk_gains=False, gain_suffix=".norm", values_are_keys=False, distance_bias=None,
                     bias_name="rel", learned_sink=False, sink_name="sink", gate_per_head=False, biases=False,
-                    bias_suffix=".b", differential=None, difference_names=DIFFERENCE_NAMES, **_) -> Dict[str, ParamSpec]:
+                    bias_suffix=".b", differential=None, difference_names=DIFFERENCE_NAMES, output_bias=True,
+                    norm_whole=False, value_mix=None, value_mix_name="vmix", **_) -> Dict[str, ParamSpec]:
         q, k, v, o, g = names
         maps = 1 if differential is None else 2
         specs = {
@@ -166,11 +186,13 @@ class BiasedAttention:
         if output_gate:
             specs[g] = ParamSpec((q_heads if gate_per_head else q_heads * value_dim, hidden_size))
         if biases:
-            for name in (q, k, o) + (() if values_are_keys else (v,)):
+            for name in (q, k) + ((o,) if output_bias else ()) + (() if values_are_keys else (v,)):
                 specs[name + bias_suffix] = ParamSpec((specs[name].shape[0],), "unit")
         if qk_gains:
-            specs[q + gain_suffix] = ParamSpec((key_dim,), "norm")
-            specs[k + gain_suffix] = ParamSpec((key_dim,), "norm")
+            specs[q + gain_suffix] = ParamSpec((q_heads * key_dim if norm_whole else key_dim,), "norm")
+            specs[k + gain_suffix] = ParamSpec((kv_heads * key_dim if norm_whole else key_dim,), "norm")
+        if value_mix is not None:
+            specs[value_mix_name] = ParamSpec((), "unit")
         if distance_bias is not None:
             specs[bias_name] = ParamSpec((int(distance_bias[0]), q_heads), "unit")
         if learned_sink:
@@ -192,7 +214,7 @@ class BiasedAttention:
             self.in_bias = torch.cat([t[n + self.bias_suffix].to(torch.float32) for n in names]).contiguous()
             if self.defer_output_bias:
                 self.deferred_bias = t[o + self.bias_suffix].to(torch.float32).contiguous()
-            else:
+            elif self.output_bias:
                 self.out_bias = t[o + self.bias_suffix].contiguous()
         if self.qk_gains:
             self.q_gain = t[q + self.gain_suffix].to(self.dtype).contiguous()
@@ -205,6 +227,8 @@ class BiasedAttention:
             self.bias_table = rel[index].t().contiguous()
         if self.learned_sink:
             self.sink_logits = t[self.sink_name].to(torch.float32).contiguous()
+        if self.value_mix == "mix":
+            self.value_share = float(t[self.value_mix_name].to(torch.float32))
         if self.differential is not None:
             diff, eps = self.differential
             a, b, c, d = (t[n].to(torch.float32) for n in self.difference_names)
@@ -227,6 +251,23 @@ class BiasedAttention:
         width_in = (self.q_heads + self.kv_heads) * self.maps * self.dk + (self.kv_heads + 2 * self.q_heads) * self.dv
         return tokens * (width_in + self.q_heads * self.maps * self.dk)
 
+    def kept_floats(self, tokens: int) -> int:
+        """What outlives the part within a step: the projections whose values later layers mix into theirs."""
+        return tokens * self.w_in.shape[0] if self.value_mix == "first" and self.w_in is not None else 0
+
+    def _value_mix(self, proj: torch.Tensor, ctx):
+        """The operand of the norm kernel: another layer's values, their bias and the share of them."""
+        if self.value_mix is None:
+            return None
+        at, n = (self.q_heads + self.kv_heads) * self.maps * self.dk, self.kv_heads * self.dv
+        if self.value_mix == "first":
+            ctx.memo[self.FIRST_VALUES] = (proj[:, at:at + n], None if self.in_bias is None else self.in_bias[at:at + n])
+            return None
+        first = ctx.memo.get(self.FIRST_VALUES)
+        if first is None:
+            raise ValueError("no layer before this one has left its values to be mixed in")
+        return first + (self.value_share,)
+
     # ---- one step
     def forward(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
         tokens = x.shape[0]
@@ -238,7 +279,8 @@ class BiasedAttention:
                            cache.page_size, self.q_heads, self.kv_heads, dk, self.dv,
                            self.unit_norm_eps, q_gain=self.q_gain, k_gain=self.k_gain, store=cache.writes,
                            inv_freq=self.inv_freq, rot_dims=self.rot_dims, q_temperature=self.q_temperature,
-                           values_are_keys=self.values_are_keys, bias=self.in_bias)
+                           values_are_keys=self.values_are_keys, bias=self.in_bias, norm_whole=self.norm_whole,
+                           rot_pairs=self.rot_pairs, value_mix=self._value_mix(proj, ctx))
         gate = None
         if self.output_gate:
             at = (self.q_heads + self.kv_heads) * dk + (0 if self.values_are_keys else self.kv_heads * self.dv)

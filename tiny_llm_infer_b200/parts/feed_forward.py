@@ -1,6 +1,6 @@
 """Dense gated feed-forward: d = (act(x Wg^T) * (x Wu^T)) Wd^T, no biases, act in float32:
 silu(g) = g / (1 + exp(-g)) (SwiGLU; reference: model/src/qwen3_paged_batch.cpp:281-295,
-kernels/src/swiglu_kernel_cpu.cpp:20-24) or, by the ``activation`` parameter, the tanh form of GELU or the clamped
+kernels/src/swiglu_kernel_cpu.cpp:20-24) or, by the ``activation`` parameter, the tanh form of GELU, ReLU or the clamped
 swish, g sigmoid(slope g) (u + 1) with g = min(gate, limit) and u = up held within -limit .. limit (``act_consts`` =
 (limit, slope)).
 ``names`` are the checkpoint's names of the gate, up and down matrices behind the part's prefix.  Gate and up projections are one product with

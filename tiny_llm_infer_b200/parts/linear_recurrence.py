@@ -1,8 +1,8 @@
 """Mixers whose memory is a matrix S [dk, dv] per (request, head) that every token decays and writes to without
 the delta rule's correction: S <- decay S + k (w v)^T, o = S^T q.  They share the scan kernel of the delta rule
 (``ops.linear_recurrence``); the state is float32, zeroed at admission and carried from step to step, so a prompt
-may come in portions of any size.  For the row's input x, with q = x Wq^T times dk^(-1/2), k = x Wk^T (heads x dk)
-and v = x Wv^T (heads x dv):
+may come in portions of any size.  For the row's input x, with q = x Wq^T times ``q_scale`` (dk^(-1/2) unless said
+otherwise), k = x Wk^T (heads x dk) and v = x Wv^T (heads x dv):
 
 ``gated_linear``   a decay per key channel, alpha = sigmoid(z)^(1/tau) with z = (x Wa1^T) Wa2^T + bias (a low rank),
                    w = 1.  The read-out is divided by its root mean square per head (``norm_eps``), times a weight of
@@ -15,8 +15,12 @@ and v = x Wv^T (heads x dv):
                    ``floor_eps``).  The read-out is divided by its root mean square per head, times a weight of
                    heads x dv numbers, times sigmoid(x Wg^T).
 
-Both end with the output product Wo.  Products: one for q | k | v | gate; one for the gates' logits (float32
-result; ``gated_linear``: the low rank first); the output.
+``fixed_decay``    q, k and v through SiLU first (``input_act``), q_scale 1; one constant decay per head (``decays``),
+                   w = 1.  The read-out of all heads together is divided by its root mean square, times a weight of
+                   heads x dv numbers, times sigmoid(x Wg^T).
+
+All end with the output product Wo.  Products: one for q | k | v | gate; one for the gates' logits, where there are
+any (float32 result; ``gated_linear``: the low rank first); the output.
 """
 from __future__ import annotations
 
@@ -149,4 +153,44 @@ class MatrixMemory(_LinearRecurrence):
                                     self.gate_act, self.out_weight, True, self.norm_eps, ctx.token_slot, ctx.seg_info,
                                     cache.state, self.heads, self.dk, self.dv, self.dk ** -0.5, self.dtype,
                                     floor_eps=self.floor_eps)
+        return ops.linear(out, self.w_o, out_dtype=self.dtype)
+
+
+@register("mixer", "fixed_decay")
+class FixedDecayAttention(_LinearRecurrence):
+    KIND = "fixed_decay"
+    NAMES = ("q", "k", "v", "g", "o", "norm")
+
+    def __init__(self, hidden_size: int, heads: int, key_dim: int, value_dim: int, decays: Sequence[float], norm_eps: float,
+                 dtype: torch.dtype, device, q_scale: float = 1.0, input_act: Optional[str] = "silu",
+                 gate_act: str = "sigmoid", names: Sequence[str] = NAMES):
+        self._init_common(hidden_size, heads, key_dim, value_dim, norm_eps, dtype, device)
+        if len(decays) != heads:
+            raise ValueError(f"{len(decays)} decays for {heads} heads")
+        if input_act not in ops.INPUT_ACTS:
+            raise ValueError(f"input activation {input_act!r}; known: {sorted(a or 'none' for a in ops.INPUT_ACTS)}")
+        self.decays = torch.tensor([float(a) for a in decays], dtype=torch.float64).to(torch.float32).to(device)
+        self.q_scale, self.input_act, self.gate_act, self.names = float(q_scale), input_act, gate_act, tuple(names)
+
+    @classmethod
+    def param_specs(cls, hidden_size, heads, key_dim, value_dim, names=NAMES, **_) -> Dict[str, ParamSpec]:
+        q, k, v, g, o, norm = names
+        qk, vd = heads * key_dim, heads * value_dim
+        return {q: ParamSpec((qk, hidden_size)), k: ParamSpec((qk, hidden_size)), v: ParamSpec((vd, hidden_size)),
+                g: ParamSpec((vd, hidden_size)), o: ParamSpec((hidden_size, vd)), norm: ParamSpec((vd,), "norm")}
+
+    def load(self, t: Dict[str, torch.Tensor]) -> None:
+        q, k, v, g, o, norm = self.names
+        self.w_in = self._pad_rows([t[q], t[k], t[v], t[g]])
+        self.out_weight = t[norm].to(torch.float32).contiguous()
+        self.w_o = t[o].contiguous()
+
+    def forward(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
+        self._check_state(cache)
+        proj = ops.linear(x, self.w_in, out_dtype=self.dtype)
+        at = self.heads * (2 * self.dk + self.dv)
+        out = ops.linear_recurrence(proj, self.KIND, None, self.decays, 1.0, proj[:, at:at + self.heads * self.dv],
+                                    self.gate_act, self.out_weight, True, self.norm_eps, ctx.token_slot, ctx.seg_info,
+                                    cache.state, self.heads, self.dk, self.dv, self.q_scale, self.dtype,
+                                    input_act=self.input_act, norm_whole=True)
         return ops.linear(out, self.w_o, out_dtype=self.dtype)
