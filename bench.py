@@ -446,6 +446,30 @@ class _DesignHarness:
             out.append(a.elapsed_time(b))
         return statistics.median(out)
 
+    def context_for(self, segs):
+        """The step context of portions (slot, first position, tokens), as the runner lays it out."""
+        import torch
+        from tiny_llm_infer_b200.engine.batch import StepContext
+        device = self.device
+        seg, tiles, dec, row = [], [], [], 0
+        for s, (slot, p0, n) in enumerate(segs):
+            seg.append([slot, row, n, p0])
+            if n == 1:
+                dec.append(row)
+            else:
+                tiles += [(s, off) for off in range(0, n, 64)]
+            row += n
+        tiles.sort(key=lambda t: (t[1] % 256 != 0, t[1] % 128 != 0))
+        pos = torch.tensor([p0 + i for _, p0, n in segs for i in range(n)], dtype=torch.int32, device=device)
+        slot = torch.tensor([sl for sl, _, n in segs for _ in range(n)], dtype=torch.int32, device=device)
+        return StepContext(tokens=row, token_ids=None, positions=pos, token_slot=slot, want_rows=None, segments=[],
+                           seg_info=torch.tensor(seg, dtype=torch.int32, device=device),
+                           dec_rows=None if len(dec) == row else torch.tensor(dec, dtype=torch.int32, device=device),
+                           n_dec=len(dec), pf_tiles=torch.tensor(tiles, dtype=torch.int32, device=device).view(-1, 2),
+                           n_tiles=len(tiles), n_tiles128=sum(1 for t in tiles if t[1] % 128 == 0),
+                           n_tiles256=sum(1 for t in tiles if t[1] % 256 == 0), max_context=self.context,
+                           max_segment=max(n for _, _, n in segs))
+
     def run_model(self, cfg, name, params, kv_bytes_per_token, state_bytes_per_request=0):
         """``params``: weights a prefill multiplies with per token (``active``) and weights a decode step reads
         (``read``); ``kv_bytes_per_token``: cache bytes a decode row reads per token of its context;
@@ -1443,7 +1467,6 @@ def vigonex_bench(args) -> int:
     from tiny_llm_infer_b200 import ops
     from tiny_llm_infer_b200.config.panolorn import (AttentionMixerConfig, FeedForwardConfig, PanolornConfig,
                                                       PanolornLayerConfig)
-    from tiny_llm_infer_b200.engine.batch import StepContext
     from tiny_llm_infer_b200.parts.registry import lookup
     from tiny_llm_infer_b200.parts.spec import PartSpec
 
@@ -1534,26 +1557,7 @@ def vigonex_bench(args) -> int:
     kern["kaketar_embedding_positions"] = hbm(per * (2 + 2 + 4), timed(lambda: ops.embedding_norm(ids, emb, h, 2.0, pos, ptab)))
     del x, h, delta, gate, out, emb, ptab
 
-    rows, page, ctx_len = 64, 16, context
-
-    def context_for(segs):
-        seg, tiles, dec, row = [], [], [], 0
-        for s, (slot, p0, n) in enumerate(segs):
-            seg.append([slot, row, n, p0])
-            if n == 1:
-                dec.append(row)
-            else:
-                tiles += [(s, off) for off in range(0, n, 64)]
-            row += n
-        tiles.sort(key=lambda t: (t[1] % 256 != 0, t[1] % 128 != 0))
-        pos = torch.tensor([p0 + i for _, p0, n in segs for i in range(n)], dtype=torch.int32, device=device)
-        slot = torch.tensor([sl for sl, _, n in segs for _ in range(n)], dtype=torch.int32, device=device)
-        return StepContext(tokens=row, token_ids=None, positions=pos, token_slot=slot, want_rows=None, segments=[],
-                           seg_info=torch.tensor(seg, dtype=torch.int32, device=device),
-                           dec_rows=None if len(dec) == row else torch.tensor(dec, dtype=torch.int32, device=device),
-                           n_dec=len(dec), pf_tiles=torch.tensor(tiles, dtype=torch.int32, device=device).view(-1, 2),
-                           n_tiles=len(tiles), n_tiles128=sum(1 for t in tiles if t[1] % 128 == 0),
-                           n_tiles256=sum(1 for t in tiles if t[1] % 256 == 0), max_context=ctx_len, max_segment=max(n for _, _, n in segs))
+    rows, page, ctx_len, context_for = 64, 16, context, hx.context_for
 
     # attention with two maps of 64 per head over values of 128, beside Panolorn's capped attention of 128 (the same
     # cache bytes; the same multiplications of queries with keys, twice those of weights with values)
@@ -1655,6 +1659,185 @@ def vigonex_bench(args) -> int:
     return 0
 
 
+SOZAVIK_SIZES = {
+    # width, layers, vocabulary and feed-forward width of the other designs' sizes; heads as Panolorn's (a_*), a recurrent
+    # state per head as Kaketar's (r_*); a window as wide as Panolorn's chunk
+    "1b": dict(width=2048, layers=8, vocab=32768, a_heads=16, a_kv=4, a_dim=128, a_vdim=128, r_heads=16, r_dim=128, ff=6144, window=2048),
+    "8b": dict(width=4096, layers=4, vocab=32768, a_heads=32, a_kv=8, a_dim=128, a_vdim=128, r_heads=32, r_dim=128, ff=12288, window=4096),
+}
+
+
+def _sozavik_at(z):
+    from tiny_llm_infer_b200.config.sozavik import (DenseConfig, FrequencyScaling, LightningConfig, RotatedAttentionConfig,
+                                                     SozavikConfig, SozavikLayerConfig, WholeNormAttentionConfig)
+    d = z["a_dim"]
+    att = RotatedAttentionConfig(z["a_heads"], z["a_kv"], d, z["a_vdim"], d ** -0.5, 50.0, z["window"], 500000.0, d // 2,
+                                 FrequencyScaling(8.0, 1.0, 4.0, 8192.0), True)
+    att2 = WholeNormAttentionConfig(z["a_heads"], z["a_kv"], d, z["a_vdim"], d ** -0.5, z["window"], True)
+    rec = LightningConfig(z["r_heads"], z["r_dim"], z["r_dim"], tuple(math.exp(-2.0 ** (-8.0 * (h + 1) / z["r_heads"]))
+                                                                      for h in range(z["r_heads"])))
+    kinds = [("attention", att), ("attention_2", att2), ("lightning", rec), ("attention_2", att2)]
+    return SozavikConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-6, logit_softcap=30.0, layers=tuple(
+        SozavikLayerConfig(*kinds[i % 4], DenseConfig(z["ff"])) for i in range(z["layers"])))
+
+
+def sozavik_bench(args) -> int:
+    """``--design sozavik``: prefill and decode throughput of the Sozavik design at sizes that resemble a real model's
+    layers (random weights, bfloat16; layers in the order rotated attention, attention normed over all heads, recurrence,
+    attention normed over all heads; dense feed-forwards), beside the closest models the engine has at equal width,
+    layers, heads, feed-forward and vocabulary, through the same step function: Panolorn (capped attention, dense) and
+    Kaketar (three delta-rule layers in four, dense).  Then the design's kernels one by one beside their relatives, with
+    their share of the measured peaks.  One JSON line."""
+    import torch
+    from tiny_llm_infer_b200 import ops
+    from tiny_llm_infer_b200.config.panolorn import (AttentionMixerConfig, FeedForwardConfig, PanolornConfig,
+                                                      PanolornLayerConfig)
+
+    hx = _DesignHarness(args)
+    device, pk, clocks, windows = hx.device, hx.pk, hx.clocks, hx.windows
+    tokens_pf, batch, context, steps, warmup = hx.tokens_pf, hx.batch, hx.context, hx.steps, hx.warmup
+    timed, run_model, context_for = hx.timed, hx.run_model, hx.context_for
+    record = {"sizes": {}}
+    for size_name in ([args.model] if args.model in SOZAVIK_SIZES else sorted(SOZAVIK_SIZES)):
+        z = SOZAVIK_SIZES[size_name]
+        W, H, G, D = z["width"], z["a_heads"], z["a_kv"], z["a_dim"]
+        pcfg = PanolornConfig(vocab=z["vocab"], width=W, embedding_scale=math.sqrt(W), norm_eps=1e-5, layers=tuple(
+            PanolornLayerConfig("attention", AttentionMixerConfig(H, G, D, D, 1.0 / math.sqrt(D), 50.0, z["window"]),
+                                FeedForwardConfig("dense", z["ff"])) for i in range(z["layers"])))
+        entry = {"config": z, "params": {}}
+        for label, cfg in (("sozavik", _sozavik_at(z)), ("panolorn", pcfg), ("kaketar", _kaketar_at(KAKETAR_SIZES[size_name]))):
+            print(f"[bench] design sizes {size_name}: {label}", file=sys.stderr, flush=True)
+            params, kvb, st = _model_costs(cfg, context)
+            head = z["vocab"] * W             # an untied embedding is a look-up; the head runs for the wanted rows alone
+            params = {"active": params - head * (2 if label != "panolorn" else 1), "read": params - (head if label != "panolorn" else 0)}
+            r = run_model(cfg, f"{label} {size_name}", params, kvb, st)
+            r["prefill_frac_of_measured"] = round(r["prefill_tflops"] / pk["bf16_tflops"], 4)
+            r["decode_hbm_frac_of_measured"] = round(r["decode_gbs"] / pk["hbm_gbs"], 4)
+            print(f"[bench] {r}", file=sys.stderr, flush=True)
+            entry[label] = r
+            entry["params"][label] = params
+        record["sizes"][size_name] = entry
+
+    # ---- kernels one by one at the larger sizes (L2 flushed between runs)
+    z = SOZAVIK_SIZES["8b"]
+    W, bf, T = z["width"], torch.bfloat16, tokens_pf
+    kern = {}
+
+    def hbm(nbytes, ms):
+        return {"us": round(ms * 1e3, 1), "gbs": round(nbytes / ms / 1e6, 1), "frac_hbm": round(nbytes / ms / 1e6 / pk["hbm_gbs"], 3)}
+
+    def tensor(flops, ms):
+        return {"us": round(ms * 1e3, 1), "tflops": round(flops / ms / 1e9, 1), "frac_tensor": round(flops / ms / 1e9 / pk["bf16_tflops"], 3)}
+
+    # norm of an output added to the stream, beside the sums with a norm of the other arrangements
+    n = 4 * T
+    h, delta = torch.randn(n, W, device=device), torch.randn(n, W, device=device).to(bf)
+    gain, out = torch.ones(W, device=device, dtype=bf), torch.empty(n, W, device=device, dtype=bf)
+    per = n * W
+    kern["stream_add_normed"] = hbm(per * (8 + 2 + 2), timed(lambda: ops.stream_add(h, delta, out, post_gain=gain, post_eps=1e-6)))
+    kern["postnorm_add_rmsnorm"] = hbm(per * (8 + 2 + 2), timed(lambda: ops.add_rmsnorm(h, delta, gain, 1e-5, out, post_gain=gain, post_eps=1e-5)))
+    kern["stream_add_normed_64_rows"] = {"us": round(timed(lambda: ops.stream_add(h[:64], delta[:64], out[:64], post_gain=gain, post_eps=1e-6)) * 1e3, 1)}
+    kern["postnorm_add_rmsnorm_64_rows"] = {"us": round(timed(lambda: ops.add_rmsnorm(
+        h[:64], delta[:64], gain, 1e-5, out[:64], post_gain=gain, post_eps=1e-5)) * 1e3, 1)}
+    del h, delta, out
+
+    rows, page, ctx_len = 64, 16, context
+    H, G, D = z["a_heads"], z["a_kv"], z["a_dim"]
+    n_pages = rows * ctx_len // page
+    table = torch.arange(n_pages, dtype=torch.int32, device=device).view(rows, ctx_len // page).contiguous()
+    pool = (torch.randn(n_pages, 2 * G * page * D, device=device) * 0.5).to(bf)
+    k_plane = pool[:, :G * page * D].unflatten(1, (G, page, D))
+    v_plane = pool[:, G * page * D:].unflatten(1, (G, page, D))
+    qk = (H + G) * D
+    in_bias, inv_freq = torch.randn(qk + G * D, device=device), torch.rand(D // 4, device=device)
+    slopes, sinks = torch.rand(H, device=device) * 0.01, torch.randn(H, device=device)
+    g1 = torch.ones(D, device=device, dtype=bf)
+    gq, gk = torch.ones(H * D, device=device, dtype=bf), torch.ones(G * D, device=device, dtype=bf)
+    for what, segs in (("prefill_2048", [(0, 0, T)]), ("decode_64_rows_ctx_2048", [(i, ctx_len - 1, 1) for i in range(rows)])):
+        ctx = context_for(segs)
+        n = ctx.tokens
+        q = torch.randn(n, H * D, device=device).to(bf)
+        o = torch.empty_like(q)
+        proj = torch.randn(n, qk + G * D + H * D, device=device).to(bf)
+        full_gate, head_gate = proj[:, qk + G * D:], proj[:, qk + G * D:qk + G * D + H]
+        other = torch.randn(n, qk + G * D, device=device).to(bf)[:, qk:]
+        moved = n * 2 * (qk + G * D) * 2
+        store = lambda eps, **more: timed(lambda: ops.qkv_unit_store(
+            proj, q, ctx.positions, ctx.token_slot, table, k_plane, v_plane, page, H, G, D, D, eps, **more))
+        kern[f"qkv_store_head_norm_pairs_bias_mix_{what}"] = hbm(moved + n * G * D * 2, store(
+            1e-6, q_gain=g1, k_gain=g1, inv_freq=inv_freq, rot_dims=D // 2, rot_pairs=True, bias=in_bias,
+            value_mix=(other, in_bias[qk:], 0.4)))
+        kern[f"qkv_store_whole_norm_mix_{what}"] = hbm(moved + n * G * D * 2, store(
+            1e-6, q_gain=gq, k_gain=gk, norm_whole=True, value_mix=(other, None, 0.4)))
+        kern[f"tetodra_qkv_store_gains_rotation_{what}"] = hbm(moved, store(1e-6, q_gain=g1, k_gain=g1, inv_freq=inv_freq, rot_dims=D // 2))
+        kern[f"panolorn_qkv_store_unit_{what}"] = hbm(moved, store(1e-6))
+        attend = lambda **more: timed(lambda: ops.attention_biased(
+            q, k_plane, v_plane, ctx.positions, ctx.token_slot, table, page, H, G, D, D, D ** -0.5, o, ctx=ctx, **more))
+        for name, ms in (("attention_cap_window_sink_head_gate", attend(softcap=50.0, window=z["window"], sink=True, sink_logits=sinks,
+                                                                        gate=head_gate, gate_per_head=True)),
+                         ("attention_window", attend(window=z["window"])),
+                         ("panolorn_attention_cap_slopes_gate", attend(softcap=50.0, chunk=4096, sink=True, slopes=slopes, gate=full_gate)),
+                         ("tetodra_attention_plain", attend())):
+            kern[f"{name}_{what}"] = tensor(2.0 * H * 2 * D * T * (T + 1) / 2, ms) if what.startswith("prefill") else \
+                hbm(rows * ctx_len * 2 * G * D * 2, ms)
+    del pool, k_plane, v_plane
+
+    # the recurrence with constant decays beside Tetodra's gated linear attention (a decay per channel) and Kaketar's delta
+    # rule, at equal state: 2048 tokens of one request, and 64 one-token rows (state read and written once per row)
+    Hr, dr = z["r_heads"], z["r_dim"]
+    inner = Hr * dr
+    words = ops.linear_recurrence_state_floats("fixed_decay", Hr, dr, dr)
+
+    def scan_record(n, ms, io, work):
+        total = io + work + (0 if n == T else 2 * rows * words * 4)
+        return {"us": round(ms * 1e3, 1), "tokens_per_s": round(n / ms * 1e3, 1), "gbs": round(total / ms / 1e6, 1),
+                "frac_hbm": round(total / ms / 1e6 / pk["hbm_gbs"], 3)}
+
+    for what, n, seg in (("prefill_2048", T, [[0, 0, T, 0]]), ("decode_64_rows", rows, None)):
+        slots = torch.zeros(n, dtype=torch.int32, device=device) if seg else torch.arange(n, dtype=torch.int32, device=device)
+        seg_info = torch.tensor(seg, dtype=torch.int32, device=device) if seg else None
+        state = torch.zeros(rows, words, device=device)
+        proj = torch.randn(n, 4 * inner, device=device).to(bf)
+        gate, zz, zb = proj[:, 3 * inner:], torch.randn(n, inner, device=device), torch.randn(inner, device=device)
+        decays, w1, wh = torch.full((Hr,), 0.99, device=device), torch.ones(dr, device=device), torch.ones(inner, device=device)
+        common = (slots, seg_info, state, Hr, dr, dr)
+        ms = timed(lambda: ops.linear_recurrence(proj, "fixed_decay", None, decays, 1.0, gate, "sigmoid", wh, True, 1e-6, *common, 1.0, bf,
+                                                 input_act="silu", norm_whole=True))
+        kern[f"fixed_decay_{what}"] = scan_record(n, ms, n * inner * (4 * 2 + 2), n * 4 * inner * 4 * 2)
+        ms = timed(lambda: ops.linear_recurrence(proj, "channel_decay", zz, zb, 1.0 / 16, gate, "silu", w1, False, 1e-6, *common, 0.1, bf))
+        kern[f"tetodra_gated_linear_{what}"] = scan_record(n, ms, n * inner * (4 * 2 + 4 + 2), n * 5 * inner * 4 * 2)
+        del state
+        taps = 4
+        state = torch.zeros(rows, ops.delta_rule_state_floats(Hr, Hr, dr, dr, taps), device=device)
+        proj = torch.randn(n, 3 * inner + Hr, device=device).to(bf)
+        conv_w = (torch.randn(3 * inner, taps, device=device) * 0.5).to(bf)
+        conv_t, rate = conv_w.t().contiguous(), torch.ones(Hr, device=device)
+        second = torch.randn(n, 2 * inner, device=device)
+        ms = timed(lambda: ops.delta_rule(proj, conv_w, taps, second[:, :inner], zb, rate, second[:, inner:], w1, 1e-6, slots, seg_info,
+                                          state, Hr, Hr, dr, dr, dr ** -0.5, 1e-6, bf, conv_t=conv_t))
+        kern[f"kaketar_delta_rule_{what}"] = scan_record(n, ms, n * inner * (3 * 2 + 2 * 4 + 2), n * 5 * inner * 4 * 2)
+        del state
+
+    # gated units: ReLU beside SiLU
+    F = z["ff"]
+    w = (torch.randn(2 * F, W, device=device) * 0.02).to(bf)
+    for n in (8, 8192):
+        xx = torch.randn(n, W, device=device).to(bf)
+        for act in ("relu", "silu"):
+            ms = timed(lambda: ops.linear_swiglu(xx, w, bf, interleaved=True, act=act))
+            kern[f"gate_up_{act}_{n}_rows"] = hbm(2 * F * W * 2, ms) if n == 8 else tensor(2.0 * n * 2 * F * W, ms)
+    ops.check_error_word(device)
+    record["kernels"] = kern
+    clock_record = clocks.stop(windows)
+    first = record["sizes"][sorted(record["sizes"])[0]]["sozavik"]
+    print(json.dumps({"metric": f"decode tok/s @ batch {batch} (Sozavik design sizes, context {context}, 1 B200)",
+                      "value": first["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": warmup,
+                      "ms_per_step": first["decode_ms"], "higher_is_better": True, "dtype": "bf16", "data": "synthetic",
+                      "design": "sozavik", "clocks": clock_record, "peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"]},
+                      **record}))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1662,7 +1845,7 @@ def main() -> int:
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--batch", type=int, default=8)
-    ap.add_argument("--model", default="8b", choices=sorted(set(MODELS) | set(DESIGN_SIZES) | set(TETODRA_SIZES) | set(PEVOLORN_SIZES) | set(VIGONEX_SIZES)),
+    ap.add_argument("--model", default="8b", choices=sorted(set(MODELS) | set(DESIGN_SIZES) | set(TETODRA_SIZES) | set(PEVOLORN_SIZES) | set(VIGONEX_SIZES) | set(SOZAVIK_SIZES)),
                     help="the sizes: 8b is the benchmark configuration, 0.6b and 32b the other two the reference is quoted on")
     ap.add_argument("--layers", type=int, default=None,
                     help="fewer layers than the model has (named in the record) if memory or time needs it")
@@ -1675,7 +1858,7 @@ def main() -> int:
     ap.add_argument("--skip-check", action="store_true", help="leave out the logits check before the timed phases")
     ap.add_argument("--ref-all", action="store_true",
                     help="reference arm: its model_main --bench at batch 1, 8 and 64 instead of --batch alone")
-    ap.add_argument("--design", default=None, choices=["panolorn", "kaketar", "tetodra", "pevolorn", "vigonex"],
+    ap.add_argument("--design", default=None, choices=["panolorn", "kaketar", "tetodra", "pevolorn", "vigonex", "sozavik"],
                     help="instead of the default workload: this design's prefill and decode throughput at sizes that "
                          "resemble a real model's layers beside Qwen3 dense at equal sizes, and its kernels one by one")
     ap.add_argument("--only", default="all", choices=["all", "prefill", "decode", "e2e", "mixed", "p128"],
@@ -1686,7 +1869,7 @@ def main() -> int:
             print("bench.py: --design runs this engine on one GPU")
             return 2
         return {"kaketar": kaketar_bench, "tetodra": tetodra_bench, "pevolorn": pevolorn_bench,
-                "vigonex": vigonex_bench}.get(args.design, design_bench)(args)
+                "vigonex": vigonex_bench, "sozavik": sozavik_bench}.get(args.design, design_bench)(args)
     if args.model not in MODELS:
         ap.error(f"--model {args.model} goes with --design")
     model_name, model_sizes = MODELS[args.model]

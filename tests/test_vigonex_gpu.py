@@ -333,7 +333,7 @@ def test_delta_rule_with_removal_per_channel(case, dtype):
 
 
 @pytest.mark.parametrize("dk,dv", [(64, 96), (128, 64), (250, 40)])
-@pytest.mark.parametrize("mode", ["delta", "channel_decay", "log_gates", "state_space", "erase"])
+@pytest.mark.parametrize("mode", ["delta", "channel_decay", "log_gates", "state_space", "erase", "fixed_decay"])
 def test_scan_with_two_columns_per_thread_changes_nothing(mode, dk, dv):
     """Every recurrence of the scan kernel: portions of 48 tokens (two columns per thread at these sizes) against the same
     tokens in portions of 8 (one), bit for bit, states included."""
@@ -370,6 +370,9 @@ def test_scan_with_two_columns_per_thread_changes_nothing(mode, dk, dv):
                 o = ops.delta_rule(cut[0], conv, 1, cut[1], zb, rate, cut[2], w1, 1e-6, *common, H, H, dk, dv, 0.1, 1e-6, f32)
             elif mode == "state_space":
                 o = ops.state_space(cut[0], conv, None, 1, hb, rate, hb, wh, 1e-6, 1, *common, H, H, dk, dv, f32)
+            elif mode == "fixed_decay":
+                o = ops.linear_recurrence(cut[0], mode, None, rate, 1.0, cut[2], "sigmoid", wh, True, 1e-6, *common, H, dk, dv, 0.1, f32,
+                                          input_act="silu", norm_whole=True)
             else:
                 o = ops.linear_recurrence(cut[0], mode, cut[1], zb, 8.0, cut[2], "silu", w1, False, 1e-6, *common, H, dk, dv, 0.1, f32)
             outs.append(o.view(slots, step, -1))
