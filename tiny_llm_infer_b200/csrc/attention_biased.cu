@@ -269,7 +269,9 @@ qkv_unit_store_vec_kernel(const bf16* proj, int row_stride, const bf16* __restri
         q_whole = 1.0f / sqrtf(q_whole / (float)(q_heads * dk) + eps);
         k_whole = 1.0f / sqrtf(k_whole / (float)(kv_heads * dk) + eps);
     }
-    for (int base = warp * kPerWarp; base < normed; base += warps * kPerWarp) {
+    // with few rows a token's heads and values are dealt to gridDim.y blocks (which all make the sums over all heads)
+    const int stride = gridDim.y * warps * kPerWarp;
+    for (int base = (blockIdx.y * warps + warp) * kPerWarp; base < normed; base += stride) {
         const int head = base + grp;
         const bool is_q = head < q_heads;
         const bool active = head < normed && e0 < dk;
@@ -334,7 +336,7 @@ qkv_unit_store_vec_kernel(const bf16* proj, int row_stride, const bf16* __restri
         // values of their own, or the keys as they were projected (before their norm): 16 bytes a thread
         const int per_head = dv / 8;
         const bf16* src0 = v_from_k ? row + (size_t)q_heads * dk : row + (size_t)normed * dk;
-        for (int c = threadIdx.x; c < kv_heads * per_head; c += blockDim.x) {
+        for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < kv_heads * per_head; c += gridDim.y * blockDim.x) {
             const int g = c / per_head, j = c - g * per_head;
             bf16* dst = v_plane + page_base + ((size_t)g * page_size + in_page) * dv + j * 8;
             if (bias == nullptr && mix.first == nullptr) {
@@ -1263,8 +1265,14 @@ int tllm_qkv_unit_store(const void* proj, int row_stride, const void* q_gain, co
                      row_stride % 8 == 0 && page_stride % 8 == 0 && aligned16(proj) && aligned16(q_out) &&
                      aligned16(k_plane) && aligned16(v_plane) && aligned16(q_gain) && aligned16(k_gain) && aligned16(bias) &&
                      (mix_first == nullptr || (aligned16(mix_first) && mix_stride % 8 == 0));
+    const int sms = sm_count_cached() > 0 ? sm_count_cached() : 148;
+    auto split_of = [&](int per_warp) {               // blocks per token: up to one run of heads per warp
+        int split = 1;
+        while (split * 8 * per_warp < q_heads + kv_heads && (long long)tokens * (split + 1) <= 2LL * sms) ++split;
+        return split;
+    };
 #define STORE_VEC(GS)                                                                                             \
-    launch_pdl(kPdlQk, qkv_unit_store_vec_kernel<GS>, dim3(tokens), dim3(256), (size_t)rot_dims * sizeof(float),  \
+    launch_pdl(kPdlQk, qkv_unit_store_vec_kernel<GS>, dim3(tokens, split_of(32 / GS)), dim3(256), (size_t)rot_dims * sizeof(float),  \
                stream, (const bf16*)proj, row_stride, (const bf16*)q_gain, (const bf16*)k_gain, eps, do_norm,     \
                positions, token_slot, block_table, max_pages, page_size, (bf16*)k_plane, (bf16*)v_plane,          \
                page_stride, (bf16*)q_out, q_heads, kv_heads, dk, dv, store, inv_freq, rot_dims, rot_pairs, temp_coef, \
